@@ -92,7 +92,7 @@ class CacheGroup:
     pool: Optional[PagePool]                       # None for groups that keep no keys/values
     kv: Dict[int, torch.Tensor] = field(default_factory=dict)
     state: Dict[int, torch.Tensor] = field(default_factory=dict)
-    states: Dict[int, Dict[str, torch.Tensor]] = field(default_factory=dict)   # entry -> named float32 states
+    states: Dict[int, Dict[str, torch.Tensor]] = field(default_factory=dict)   # entry -> named states
 
     @property
     def paged(self) -> bool:
@@ -193,8 +193,8 @@ class CacheManager:
                                                 dtype=dtype, device=self.device)
                     if n.states:
                         # Not cleared when a slot is taken again: a mixer starts from zero at position 0.
-                        grp.states[e] = {name: torch.zeros((max_requests, *shape), dtype=torch.float32, device=self.device)
-                                         for name, shape in n.states}
+                        grp.states[e] = {name: torch.zeros((max_requests, *shape), dtype=kind[0] if kind else torch.float32, device=self.device)
+                                         for name, shape, *kind in n.states}
                     if n.state_shape is not None:
                         grp.state[e] = torch.zeros((max_requests, *n.state_shape),
                                                    dtype=n.state_dtype or torch.float32, device=self.device)

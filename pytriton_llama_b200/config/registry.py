@@ -64,6 +64,9 @@ def _register_builtin() -> None:
     from .podizen import PodizenConfig
     from ..models.podizen import podizen_spec
     register_architecture("Podizen", PodizenConfig.from_dict, podizen_spec)
+    from .nesisun import NesisunConfig
+    from ..models.nesisun import nesisun_spec
+    register_architecture("Nesisun", NesisunConfig.from_dict, nesisun_spec)
 
 
 _register_builtin()

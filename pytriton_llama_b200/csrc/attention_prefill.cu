@@ -12,7 +12,8 @@
 // key) off the scores of head h; `gate_col` >= 0 multiplies the result of head h by the sigmoid of the D entries at
 // column gate_col + h * D of the token's q row; `pool` = P > 0 (with a window) puts key tiles of block means in front:
 // entry b of `summary` (pages laid out as the cache's, with a block table of their own) is the mean key and mean
-// value of positions bP .. bP + P - 1, seen by the query at position p if bP + P - 1 <= p - window.
+// value of positions bP .. bP + P - 1, seen by the query at position p if bP + P - 1 <= p - window; `sink_logits` [heads]:
+// the sink's term has that score for a head instead of 0.
 //
 // tiles[i] = {request row, first token index, rows (0..128; 0: nothing to do), position of the first token}.
 #include "mma_utils.cuh"
@@ -38,6 +39,7 @@ struct PrefillExtras {
   const __nv_bfloat16* summary;
   const int* sum_bt;
   int sum_bt_stride, sum_pages;
+  const float* sink_logits;
 };
 
 // MT = 16-row tiles per warp: 2 for head size 64 (4 warps), 1 for 128 (8 warps).
@@ -287,10 +289,11 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
     for (int hh = 0; hh < 2; ++hh) {
       const int row = wrow0 + mt * 16 + g + hh * 8;
       if (row >= rows) continue;
-      if (sink) {       // one more term of score 0 and no value: the maximum may move to 0, and 2^(0 - maximum) joins the sum
-        const float m_all = fmaxf(m_run[mt][hh], 0.f);
+      if (sink) {       // one more term and no value: the maximum may move to its score z, and 2^(z - maximum) joins the sum
+        const float z = ex.sink_logits ? ex.sink_logits[h] * 1.4426950408889634f : 0.f;
+        const float m_all = fmaxf(m_run[mt][hh], z);
         const float a = exp2f(m_run[mt][hh] - m_all);
-        l_run[mt][hh] = fmaf(l_run[mt][hh], a, exp2f(-m_all));
+        l_run[mt][hh] = fmaf(l_run[mt][hh], a, exp2f(z - m_all));
 #pragma unroll
         for (int i = 0; i < D / 8; ++i) { o[mt][i][2 * hh] *= a; o[mt][i][2 * hh + 1] *= a; }
       }
@@ -314,7 +317,7 @@ template <int D, int MT>
 int launch_prefill(void* out, const void* q, const void* cache, const int* block_table, const int* tiles, int n_tiles,
                    int q_stride, int out_stride, int bt_stride, int nq, int nkv, int page_size, float scale,
                    int window, int num_pages, void* stream, int keep = 0, int sink = 0, float temp_coef = 0.f, int temp_every = 1,
-                   PrefillExtras ex = {0.f, -1, 0, nullptr, nullptr, 0, 0}) {
+                   PrefillExtras ex = {0.f, -1, 0, nullptr, nullptr, 0, 0, nullptr}) {
   using Cfg = PrefillCfg<D, MT>;
   static SmemRaised raised = {};
   if (int rc = raise_shared_memory("prefill_attention", prefill_attention_kernel<D, MT>, Cfg::kSmem, raised)) return rc;
@@ -369,20 +372,22 @@ PTL_EXPORT int ptl_prefill_attention_keep_bf16(void* out, const void* q, const v
                                 page_size, scale, window, num_pages, stream, keep);
 }
 
-// The same with the options of the window attention's other kernel: `sink` adds one term of score 0 (and no value) to
-// every softmax's denominator; `temp_coef` != 0 multiplies the scores of the query at position p by
+// The same with the options of the window attention's other kernel: `sink` adds one term of score 0, or of score
+// sink_logits[head], (and no value) to every softmax's denominator; `temp_coef` != 0 multiplies the scores of the query at position p by
 // 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).
 PTL_EXPORT int ptl_prefill_attention_opts_bf16(void* out, const void* q, const void* cache, const int* block_table,
                                                const int* tiles, int n_tiles, int q_stride, int out_stride, int bt_stride,
                                                int nq, int nkv, int d, int page_size, float scale, int window, int keep,
                                                int num_pages, int sink, float temp_coef, int temp_every, float bias_exp,
                                                int gate_col, int pool, const void* summary, const int* sum_bt, int sum_bt_stride,
-                                               int sum_pages, void* stream) {
+                                               int sum_pages, const float* sink_logits, void* stream) {
   using namespace ptl;
+  if (sink_logits) sink = 1;
   PTL_REQUIRE(pool == 0 || (summary && sum_bt && sum_pages > 0 && window > 0 && keep == 0 && !sink && aligned16(summary)),
               "prefill_attention: means of blocks need their pages and a window, and go with no kept positions or sink");
   PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || (gate_col + nq * d <= q_stride && gate_col % 2 == 0)), "prefill_attention: bad bias or gate column");
-  const PrefillExtras ex = {bias_exp, gate_col, window > 0 ? pool : 0, (const __nv_bfloat16*)summary, sum_bt, sum_bt_stride, sum_pages};
+  const PrefillExtras ex = {bias_exp, gate_col, window > 0 ? pool : 0, (const __nv_bfloat16*)summary, sum_bt, sum_bt_stride, sum_pages,
+                            sink_logits};
   PTL_REQUIRE(n_tiles >= 0 && nq > 0 && nkv > 0 && page_size > 0 && num_pages > 0 && keep >= 0 && temp_every >= 1,
               "prefill_attention: bad sizes");
   PTL_REQUIRE(nq % nkv == 0, "prefill_attention: %d query heads are no multiple of %d kv heads", nq, nkv);

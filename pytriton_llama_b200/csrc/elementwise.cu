@@ -1,4 +1,4 @@
-// Row-wise kernels: embedding gather, residual add fused with RMSNorm, SiLU(gate)*up.
+// Row-wise kernels: embedding gather, residual add fused with RMSNorm, act(gate)*up.
 // Each takes any width (no power of two needed); 16-byte packets are used when the row pitch
 // allows it, scalars otherwise.
 #include "common.cuh"
@@ -170,35 +170,35 @@ add_rmsnorm_warp_kernel(T* __restrict__ y, float* __restrict__ residual_out, con
   }
 }
 
-// ------------------------------------------------------------------ SiLU(gate) * up
-// gu is [T, 2*inter] (gate columns first); out[t, i] = g * sigmoid(g) * u in float32.
+// ------------------------------------------------------------------ act(gate) * up
+// gu is [T, 2*inter] (gate columns first); out[t, i] = act(g) * u in float32, act SiLU (`gelu` 0) or the tanh form of
+// gelu (1); rows of `out` start out_ld elements apart.
+__device__ __forceinline__ float gate_activation(float z, int gelu) {
+  if (gelu) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.0f + expf(-z));
+}
+
 template <typename T>
-__global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, int inter, int vec_ok) {
+__global__ void gated_act_kernel(T* __restrict__ out, int out_ld, const T* __restrict__ gu, int inter, int gelu, int vec_ok) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.y;
   const T* g = gu + (size_t)t * 2 * inter;
   const T* u = g + inter;
-  T* o = out + (size_t)t * inter;
+  T* o = out + (size_t)t * out_ld;
   constexpr int VN = Vec16<T>::N;
   if (vec_ok) {
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * VN;
     if (i < inter) {
       Vec16<T> a = load16(g + i), b = load16(u + i), c;
 #pragma unroll
-      for (int k = 0; k < VN; ++k) {
-        const float gv = a.get(k);
-        c.set(k, gv / (1.0f + expf(-gv)) * b.get(k));
-      }
+      for (int k = 0; k < VN; ++k) c.set(k, gate_activation(a.get(k), gelu) * b.get(k));
       store16(o + i, c);
     }
   } else {
     for (int k = 0; k < VN; ++k) {
       const int i = (blockIdx.x * blockDim.x + threadIdx.x) * VN + k;
-      if (i < inter) {
-        const float gv = to_f32(g[i]);
-        o[i] = from_f32<T>(gv / (1.0f + expf(-gv)) * to_f32(u[i]));
-      }
+      if (i < inter) o[i] = from_f32<T>(gate_activation(to_f32(g[i]), gelu) * to_f32(u[i]));
     }
   }
 }
@@ -284,16 +284,16 @@ int add_rmsnorm(void* y, float* residual_out, const float* residual_in, const vo
 }
 
 template <typename T>
-int silu_mul(void* out, const void* gu, int tokens, int inter, void* stream) {
-  PTL_REQUIRE(tokens >= 0 && inter > 0, "silu_mul: bad sizes tokens=%d inter=%d", tokens, inter);
-  PTL_REQUIRE(tokens <= 65535, "silu_mul: at most 65535 rows per call, got %d", tokens);
+int gated_act(void* out, int out_ld, const void* gu, int tokens, int inter, int gelu, void* stream) {
+  PTL_REQUIRE(tokens >= 0 && inter > 0 && out_ld >= inter, "gated_act: bad sizes tokens=%d inter=%d out_ld=%d", tokens, inter, out_ld);
+  PTL_REQUIRE(tokens <= 65535, "gated_act: at most 65535 rows per call, got %d", tokens);
   if (tokens == 0) return 0;
   constexpr int VN = Vec16<T>::N;
-  const int vec_ok = (inter % VN == 0) && aligned16(out) && aligned16(gu);
+  const int vec_ok = (inter % VN == 0) && (out_ld % VN == 0) && aligned16(out) && aligned16(gu);
   const int threads = 256;
   dim3 grid((inter + threads * VN - 1) / (threads * VN), tokens);
-  return launch_kernel("silu_mul", silu_mul_kernel<T>, grid, dim3(threads), 0, as_stream(stream), (T*)out, (const T*)gu,
-                       inter, vec_ok);
+  return launch_kernel("gated_act", gated_act_kernel<T>, grid, dim3(threads), 0, as_stream(stream), (T*)out, out_ld, (const T*)gu,
+                       inter, gelu, vec_ok);
 }
 
 }  // namespace ptl
@@ -364,9 +364,9 @@ PTL_EXPORT int ptl_add_bias_rmsnorm_f32(void* y, float* residual_out, const floa
 PTL_EXPORT int ptl_add_bias_rmsnorm_bf16(void* y, float* residual_out, const float* residual_in, const void* x, const float* bias, const float* w, const int* rows, int out_rows, int hidden, float eps, void* stream) {
   return ptl::add_rmsnorm<__nv_bfloat16>(y, residual_out, residual_in, x, w, rows, out_rows, hidden, eps, stream, bias);
 }
-PTL_EXPORT int ptl_silu_mul_f32(void* out, const void* gu, int tokens, int inter, void* stream) {
-  return ptl::silu_mul<float>(out, gu, tokens, inter, stream);
+PTL_EXPORT int ptl_gated_act_f32(void* out, int out_ld, const void* gu, int tokens, int inter, int gelu, void* stream) {
+  return ptl::gated_act<float>(out, out_ld, gu, tokens, inter, gelu, stream);
 }
-PTL_EXPORT int ptl_silu_mul_bf16(void* out, const void* gu, int tokens, int inter, void* stream) {
-  return ptl::silu_mul<__nv_bfloat16>(out, gu, tokens, inter, stream);
+PTL_EXPORT int ptl_gated_act_bf16(void* out, int out_ld, const void* gu, int tokens, int inter, int gelu, void* stream) {
+  return ptl::gated_act<__nv_bfloat16>(out, out_ld, gu, tokens, inter, gelu, stream);
 }

@@ -65,7 +65,8 @@ PTL_EXPORT int ptl_gemm_tc_k_parts(int M, int N, int K) {
   return plan_tiles(M, N, K, true).parts;
 }
 
-// out: epi 0 bf16 [M,N]; 1 float32 [M,N]; 2 float32 [M,N] added to in place; 3 bf16 [M,N/2].
+// out: epi 0 bf16 [M,N]; 1 float32 [M,N]; 2 float32 [M,N] added to in place; 3 bf16 [M,N/2], silu(gate) * up of weight
+// rows that alternate gate, up; 5 the same with the tanh form of gelu.
 // Returns -2 when the sizes are not ones this kernel takes (K % 8 != 0 or K < 64), so that the caller
 // can use another product.  `splits_hint` > 0 forces the number of K splits when M <= 64 (1, 2, 4 or 8);
 // when M > 64 it asks for that many parts of the K range, whose partial sums are stored one after
@@ -87,9 +88,15 @@ static int gemm_tc_impl(void* out, const void* X, const void* W, int M, int N, i
   PTL_REQUIRE(M >= 0 && N > 0 && K > 0 && ld_out > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
   if (K % 8 != 0 || K < kTileK) return -2;
   PTL_REQUIRE(aligned16(X) && aligned16(W) && aligned16(out), "gemm_tc: operands must be 16-byte aligned");
-  PTL_REQUIRE(epi != 3 || N % 2 == 0, "gemm_tc: the SiLU*up epilogue needs an even number of weight rows");
-  if (M == 0) return 0;
   GemmParams p{};
+  p.gate_a = 1.0f;
+  if (epi == 5) {
+    epi = 3;
+    p.gate_a = 1.5957691216057308f;      // 2 sqrt(2 / pi)
+    p.gate_b = 0.044715f * p.gate_a;
+  }
+  PTL_REQUIRE(epi != 3 || N % 2 == 0, "gemm_tc: the gate*up epilogue needs an even number of weight rows");
+  if (M == 0) return 0;
   p.out = out; p.status = status;
   p.K = K; p.ld_out = ld_out;
   p.poll_limit = poll_limit; p.withhold_first_load = withhold_first_load;
@@ -179,7 +186,7 @@ PTL_EXPORT int ptl_gemm_tc_bf16_norm(void* out, const void* X, const void* W, in
                                      int* status, int splits_hint, void* xs, const float* norm_w, float* sumsq,
                                      int sumsq_ld, int* slots_out, const float* scale_sumsq, int scale_slots,
                                      int scale_ld, float scale_eps, void* stream) {
-  PTL_REQUIRE(epi >= 0 && epi <= 3, "gemm_tc: unknown epilogue %d", epi);
+  PTL_REQUIRE((epi >= 0 && epi <= 3) || epi == 5, "gemm_tc: unknown epilogue %d", epi);
   return gemm_tc_impl(out, X, W, M, N, K, ld_out, epi, status, splits_hint, xs, norm_w, sumsq, sumsq_ld, slots_out, scale_sumsq,
                       scale_slots, scale_ld, scale_eps, nullptr, stream);
 }

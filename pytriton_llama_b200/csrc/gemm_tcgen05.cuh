@@ -80,6 +80,7 @@ struct GemmParams {
   // run out, and the test sees the status word, the drained roles and the block's clean exit.
   uint32_t poll_limit;
   int withhold_first_load;
+  float gate_a, gate_b;           // epilogue 3: the gate's activation (gate_act)
   unsigned long long* timeline;   // measurements: where the first and the last block stamp %globaltimer (null: nowhere)
   int timeline_kind;
 };
@@ -124,9 +125,12 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&t);
 }
 
-// SiLU for the bfloat16 path: the result is rounded to 8 bits of mantissa, so the fast
-// exponential and reciprocal (about 2 ulp of float32) cost no accuracy that survives.
-__device__ __forceinline__ float silu_f(float g) { return __fdividef(g, 1.0f + __expf(-g)); }
+// The gate's activation for the bfloat16 path, g * sigmoid(g * (a + b g^2)): a = 1, b = 0 is SiLU; a = 2 sqrt(2/pi),
+// b = 0.044715 a is the tanh form of gelu, since (1 + tanh(z)) / 2 = sigmoid(2z).  The result is rounded to 8 bits of
+// mantissa, so the fast exponential and reciprocal (about 2 ulp of float32) cost no accuracy that survives.
+__device__ __forceinline__ float gate_act(const GemmParams& p, float g) {
+  return __fdividef(g, 1.0f + __expf(-g * fmaf(p.gate_b, g * g, p.gate_a)));
+}
 
 // ---------------------------------------------------------------- epilogue of one row's 16 accumulators
 // Normal mode: `row` is a token, columns c0..c0+15 are features.
@@ -141,14 +145,14 @@ __device__ __forceinline__ void store_normal(const GemmParams& p, int row, int c
       uint32_t* w = reinterpret_cast<uint32_t*>(&pk);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        __nv_bfloat162 t = __floats2bfloat162_rn(silu_f(v[4 * j]) * v[4 * j + 1], silu_f(v[4 * j + 2]) * v[4 * j + 3]);
+        __nv_bfloat162 t = __floats2bfloat162_rn(gate_act(p, v[4 * j]) * v[4 * j + 1], gate_act(p, v[4 * j + 2]) * v[4 * j + 3]);
         w[j] = *reinterpret_cast<uint32_t*>(&t);
       }
       *reinterpret_cast<uint4*>(o) = pk;
     } else {
 #pragma unroll
       for (int j = 0; j < 8; ++j)
-        if (c0 + 2 * j + 1 < n_total) o[j] = __float2bfloat16_rn(silu_f(v[2 * j]) * v[2 * j + 1]);
+        if (c0 + 2 * j + 1 < n_total) o[j] = __float2bfloat16_rn(gate_act(p, v[2 * j]) * v[2 * j + 1]);
     }
     return;
   }
@@ -231,7 +235,7 @@ __device__ __forceinline__ void store_swapped(const GemmParams& p, int row, int 
     if (EPI == 3) {
       const float up = __shfl_down_sync(0xffffffffu, v[j], 1);   // odd rows hold up_j; all lanes take part
       if (n_ok && tok < p.cols && (n & 1) == 0)
-        ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n / 2] = __float2bfloat16_rn(silu_f(v[j]) * up);
+        ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n / 2] = __float2bfloat16_rn(gate_act(p, v[j]) * up);
     } else if (EPI == 2) {
       add_and_emit(p, n, tok, v[j], false, 0.f, threadIdx.x & 31);
     } else if (n_ok && tok < p.cols) {
@@ -248,7 +252,7 @@ __device__ __forceinline__ void store_swapped_one(const GemmParams& p, int n, in
   if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n] = __float2bfloat16_rn(v);
   else if (EPI == 1) ((float*)p.out)[(size_t)tok * p.ld_out + n] = v;
   else if (EPI == 2) ((float*)p.out)[(size_t)tok * p.ld_out + n] += v;
-  else ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n / 2] = __float2bfloat16_rn(silu_f(v) * up);
+  else ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n / 2] = __float2bfloat16_rn(gate_act(p, v) * up);
 }
 
 // 16 columns of this thread's TMEM lane, added over the issuers' accumulators; an issuer that had
@@ -797,10 +801,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_row, const __grid_constan
             if (col < p.cols) {
               __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)col * p.ld_out + n / 2;
               if (n + 3 < p.rows && p.ld_out % 2 == 0) {
-                *reinterpret_cast<uint32_t*>(o) = pack_bf16x2(silu_f(v[0]) * v[1], silu_f(v[2]) * v[3]);
+                *reinterpret_cast<uint32_t*>(o) = pack_bf16x2(gate_act(p, v[0]) * v[1], gate_act(p, v[2]) * v[3]);
               } else {
-                if (n + 1 < p.rows) o[0] = __float2bfloat16_rn(silu_f(v[0]) * v[1]);
-                if (n + 3 < p.rows) o[1] = __float2bfloat16_rn(silu_f(v[2]) * v[3]);
+                if (n + 1 < p.rows) o[0] = __float2bfloat16_rn(gate_act(p, v[0]) * v[1]);
+                if (n + 3 < p.rows) o[1] = __float2bfloat16_rn(gate_act(p, v[2]) * v[3]);
               }
             }
           } else if (col < p.cols) {

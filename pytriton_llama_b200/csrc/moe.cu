@@ -5,16 +5,22 @@
 //                 lower index wins a tie), expert ids and scores out.  Options: score = softmax(logit) over
 //                 all experts; `groups` > 1: experts form that many groups of neighbours, a group's score is
 //                 its largest score and only experts of the `keep` best groups can be chosen (the lower group
-//                 wins a tie); `renorm`: the chosen scores are divided by their sum + 1e-20.
+//                 wins a tie); `correction` [E]: experts are chosen by score + correction and weighted by the score
+//                 alone; `renorm`: the chosen scores are divided by their sum + 1e-20; `scale` multiplies the weights.
 //   moe_plan      one block: tokens per expert, each expert's rows padded to whole tiles of kMoeTile rows,
-//                 the list of tiles (expert, first row, rows), the row of every (token, choice).
+//                 the list of tiles (expert, first row, rows), the row of every (token, choice); -1 for a choice
+//                 whose id is at or beyond the number of experts that have weights.
 //   moe_gather    sorted[row] = x[token] (* score when the weight multiplies the expert's input), rounded to T.
 //   moe_grouped   C[row, :] = A[row, :] . W[expert]^T for the rows of a tile; either plain (float32 out) or
-//                 with W = [gate rows | up rows] and silu(gate) * up as the result (T out).  CUDA-core
+//                 with W = [gate rows | up rows] and silu(gate) * up, or with `limit` > 0 the clamped form
+//                 min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + shift), as the result (T out).  CUDA-core
 //                 form for both element types: sums run over K in ascending order in chunks of 32 that are
 //                 added to the total one by one, the same for every row wherever it lies in its tile.
 //   moe_combine   out[token] = shared[token] + sum over its choices of C[row] (times the score when the
 //                 weight multiplies the expert's output), float32.
+//   moe_combine_norm   the same with choices that have no row standing for the token's own input x (an expert without
+//                 weights hands its input on), added together with another sub-layer's output into the float32
+//                 residual, and optionally the RMS norm that reads the residual next.  One kernel.
 // A block that finds its tile index beyond the tile count returns at once: the grid is sized for the
 // most tiles a step of this many tokens can have.
 #include "common.cuh"
@@ -27,12 +33,21 @@ constexpr int kMoeWide = 128;         // rows of a wide tile (steps of many toke
 constexpr int kMoeMaxExperts = 1024;
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float moe_silu(float x) { return x / (1.0f + expf(-x)); }
+// The product of a gate and its up value: silu(g) * u, or the clamped form (limit > 0).
+struct GluForm { float limit, alpha, shift; };
+__device__ __forceinline__ float moe_glu(float g, float u, const GluForm& f) {
+  if (f.limit > 0.f) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit);
+    return g / (1.0f + expf(-f.alpha * g)) * (u + f.shift);
+  }
+  return g / (1.0f + expf(-g)) * u;
+}
 
 // ------------------------------------------------------------------ route
 __global__ void __launch_bounds__(128)
 moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits, int tokens, int E,
-                 int top, int softmax, int groups, int keep, int renorm) {
+                 int top, int softmax, int groups, int keep, int renorm, const float* __restrict__ correction, float scale) {
   __shared__ float s_best[4][kMoeMaxExperts];      // per warp: the largest score of every group
   pdl_wait();
   pdl_launch_dependents();
@@ -102,6 +117,20 @@ moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float
       }
     }
   }
+  if (correction) {          // from here on `sc` holds the choice scores; the scores themselves are kept aside for the weights
+    float* own = s_best[warp];
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      if (32 * i >= E) break;
+      const int e = lane + 32 * i;
+      if (e < E) {
+        own[e] = sc[i];
+        sc[i] += correction[e];
+        if (!(sc[i] == sc[i])) sc[i] = -INFINITY;
+      }
+    }
+    __syncwarp();
+  }
   float total = 0.f, held = 0.f;           // lane k holds the k-th chosen score (the first 32 of them)
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -119,6 +148,7 @@ moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float
       if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
     }
     if (best_e >= E) { best_e = k % E; best = 0.f; }            // nothing finite left: a valid expert with weight 0
+    else if (correction) best = fmaxf(s_best[warp][best_e], 0.f);   // the weight is the score as it was
     total += best;                                               // in the order they were chosen, the same in every lane
     if (k == lane) held = best;
     if (lane == 0) {
@@ -131,9 +161,9 @@ moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float
       if (lane + 32 * i == best_e) sc[i] = -INFINITY;
     }
   }
-  const float inv = renorm ? 1.0f / (total + 1e-20f) : 1.0f;
+  const float inv = (renorm ? 1.0f / (total + 1e-20f) : 1.0f) * scale;
   if (lane < top) weights[(size_t)t * top + lane] = held * inv;
-  if (renorm && top > 32) {
+  if (inv != 1.0f && top > 32) {
     __syncwarp();                          // lane 0's weights beyond the 32nd, read back by the others
     for (int k = 32 + lane; k < top; k += 32) weights[(size_t)t * top + k] *= inv;
   }
@@ -243,7 +273,7 @@ moe_gather_kernel(T* __restrict__ sorted, const T* __restrict__ x, const int* __
 template <typename T, typename OUT, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_grouped_kernel(OUT* __restrict__ C, int ldc, const T* __restrict__ A, const T* __restrict__ W, const int* __restrict__ tiles,
-                   const int* __restrict__ meta, int N, int K, size_t expert_stride, int half) {
+                   const int* __restrict__ meta, int N, int K, size_t expert_stride, int half, const GluForm form) {
   __shared__ float sa[kMoeTile][33], sb[64][33];
   pdl_wait();
   pdl_launch_dependents();
@@ -307,7 +337,7 @@ moe_grouped_kernel(OUT* __restrict__ C, int ldc, const T* __restrict__ A, const 
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int f = j0 + tx + 16 * j;
-        if (f < half) dst[f] = from_f32<OUT>(moe_silu(total[i][j]) * total[i][j + 2]);
+        if (f < half) dst[f] = from_f32<OUT>(moe_glu(total[i][j], total[i][j + 2], form));
       }
     } else {
 #pragma unroll
@@ -332,7 +362,7 @@ template <typename OUT, bool GATED>
 __global__ void __launch_bounds__(128)
 moe_grouped_mma_kernel(OUT* __restrict__ C, int ldc, const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __restrict__ W,
                        const int* __restrict__ tiles, const int* __restrict__ meta, int N, int K, size_t expert_stride,
-                       int half) {
+                       int half, const GluForm form) {
   extern __shared__ __align__(16) unsigned char moe_smem[];
   __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(moe_smem);
   pdl_wait();
@@ -443,7 +473,7 @@ moe_grouped_mma_kernel(OUT* __restrict__ C, int ldc, const __nv_bfloat16* __rest
           for (int e = 0; e < 4; ++e) {
             const int rr = mt * 16 + g + (e >> 1) * 8, cc = warp * 16 + nt * 8 + 2 * c + (e & 1);
             const int f = j0 + cc;
-            if (rr < rows && f < half) C[(size_t)(row0 + rr) * ldc + f] = from_f32<OUT>(moe_silu(acc[mt][nt][e]) * s_up[rr * 33 + cc]);
+            if (rr < rows && f < half) C[(size_t)(row0 + rr) * ldc + f] = from_f32<OUT>(moe_glu(acc[mt][nt][e], s_up[rr * 33 + cc], form));
           }
     }
   } else {
@@ -473,7 +503,7 @@ template <typename OUT, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_grouped_wide_kernel(OUT* __restrict__ C, int ldc, const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __restrict__ W,
                         const int* __restrict__ tiles, const int* __restrict__ meta, int N, int K, size_t expert_stride,
-                        int half) {
+                        int half, const GluForm form) {
   extern __shared__ __align__(16) unsigned char wide_smem[];
   __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(wide_smem);
   pdl_wait();
@@ -574,7 +604,7 @@ moe_grouped_wide_kernel(OUT* __restrict__ C, int ldc, const __nv_bfloat16* __res
 #pragma unroll
           for (int e1 = 0; e1 < 2; ++e1) {
             const int f = j0 + wn * 32 + nt * 8 + 2 * c + e1;
-            if (f < half) dst[f] = from_f32<OUT>(moe_silu(acc[mt][nt][2 * e2 + e1]) * acc[mt][nt + 4][2 * e2 + e1]);
+            if (f < half) dst[f] = from_f32<OUT>(moe_glu(acc[mt][nt][2 * e2 + e1], acc[mt][nt + 4][2 * e2 + e1], form));
           }
       } else {
 #pragma unroll
@@ -589,7 +619,7 @@ moe_grouped_wide_kernel(OUT* __restrict__ C, int ldc, const __nv_bfloat16* __res
 }
 
 int moe_grouped_wide(void* C, int ldc, const void* A, const void* W, const int* wide, const int* meta, int max_wide, int N, int K,
-                     int gated, void* stream) {
+                     int gated, GluForm form, void* stream) {
   PTL_REQUIRE(max_wide >= 0 && N > 0 && K > 0 && (!gated || N % 2 == 0), "moe_grouped_wide: bad sizes N=%d K=%d", N, K);
   if (K % 8 != 0 || !aligned16(A) || !aligned16(W)) return -2;
   if (max_wide == 0) return 0;
@@ -602,11 +632,11 @@ int moe_grouped_wide(void* C, int ldc, const void* A, const void* W, const int* 
   if (gated) {
     if (int rc = raise_shared_memory("moe_grouped_wide", moe_grouped_wide_kernel<B, true>, kWideSmem, raised_gated)) return rc;
     return launch_kernel("moe_grouped_wide", moe_grouped_wide_kernel<B, true>, grid, dim3(256), kWideSmem, as_stream(stream), (B*)C,
-                         ldc, (const B*)A, (const B*)W, wide, meta, N, K, stride, half);
+                         ldc, (const B*)A, (const B*)W, wide, meta, N, K, stride, half, form);
   }
   if (int rc = raise_shared_memory("moe_grouped_wide", moe_grouped_wide_kernel<float, false>, kWideSmem, raised_plain)) return rc;
   return launch_kernel("moe_grouped_wide", moe_grouped_wide_kernel<float, false>, grid, dim3(256), kWideSmem, as_stream(stream),
-                       (float*)C, ldc, (const B*)A, (const B*)W, wide, meta, N, K, stride, half);
+                       (float*)C, ldc, (const B*)A, (const B*)W, wide, meta, N, K, stride, half, form);
 }
 
 // ------------------------------------------------------------------ combine
@@ -661,15 +691,116 @@ moe_combine_kernel(float* __restrict__ out, const float* __restrict__ C, const T
   }
 }
 
+// ------------------------------------------------------------------ combine, add into the residual, next norm
+// residual[t] += add[t] (T or null) + shared[t] + sum over the choices of weight * (C[row], or x[t] where the choice has no
+// row), in float32 and in this order; with `norm_w` y[t] = residual[t] * rsqrt(mean(residual[t]^2) + eps) * norm_w.  The
+// new row is kept in shared memory between the two passes.
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+  if constexpr (sizeof(T) == 4) {
+    return *reinterpret_cast<const float4*>(p);
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_combine_norm_kernel(float* __restrict__ residual, T* __restrict__ y, const float* __restrict__ C, const T* __restrict__ x,
+                        const T* __restrict__ add, const T* __restrict__ shared_out, const int* __restrict__ pos,
+                        const float* __restrict__ weights, const float* __restrict__ norm_w, int top, int width, float eps,
+                        int vec_ok) {
+  extern __shared__ __align__(16) float row_smem[];
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int* tp = pos + (size_t)t * top;
+  const float* tw = weights + (size_t)t * top;
+  float* res = residual + (size_t)t * width;
+  const T* xr = x + (size_t)t * width;
+  const size_t base = (size_t)t * width;
+  float ss = 0.f;
+  if (vec_ok) {
+    for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+      float4 acc = *reinterpret_cast<const float4*>(res + i);
+      const float4 own = load4(xr + i);
+      if (add) { const float4 v = load4(add + base + i); acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w; }
+      if (shared_out) { const float4 v = load4(shared_out + base + i); acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w; }
+      for (int k0 = 0; k0 < top; k0 += 4) {        // four choices' rows are requested together, then added in the order of the choices
+        float4 v[4];
+        float wk[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const bool have = k0 + u < top;
+          const int row = have ? tp[k0 + u] : -1;
+          wk[u] = have ? tw[k0 + u] : 0.f;
+          v[u] = row < 0 ? own : *reinterpret_cast<const float4*>(C + (size_t)row * width + i);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          acc.x = fmaf(wk[u], v[u].x, acc.x); acc.y = fmaf(wk[u], v[u].y, acc.y);
+          acc.z = fmaf(wk[u], v[u].z, acc.z); acc.w = fmaf(wk[u], v[u].w, acc.w);
+        }
+      }
+      *reinterpret_cast<float4*>(res + i) = acc;
+      if (norm_w) {
+        *reinterpret_cast<float4*>(row_smem + i) = acc;
+        ss += acc.x * acc.x + acc.y * acc.y + acc.z * acc.z + acc.w * acc.w;
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+      float acc = res[i];
+      if (add) acc += to_f32(add[base + i]);
+      if (shared_out) acc += to_f32(shared_out[base + i]);
+      for (int k = 0; k < top; ++k) {
+        const int row = tp[k];
+        acc = fmaf(tw[k], row < 0 ? to_f32(xr[i]) : C[(size_t)row * width + i], acc);
+      }
+      res[i] = acc;
+      if (norm_w) {
+        row_smem[i] = acc;
+        ss += acc * acc;
+      }
+    }
+  }
+  if (!norm_w) return;
+  ss = block_sum(ss, red);
+  const float rrms = 1.0f / sqrtf(ss / (float)width + eps);
+  T* yo = y + (size_t)t * width;
+  if (vec_ok) {
+    for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+      const float4 s = *reinterpret_cast<const float4*>(row_smem + i);
+      const float4 g = *reinterpret_cast<const float4*>(norm_w + i);
+      const float4 o = make_float4(s.x * rrms * g.x, s.y * rrms * g.y, s.z * rrms * g.z, s.w * rrms * g.w);
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(yo + i) = o;
+      } else {
+        uint2 pk;
+        *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(o.x, o.y);
+        *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(o.z, o.w);
+        *reinterpret_cast<uint2*>(yo + i) = pk;
+      }
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) yo[i] = from_f32<T>(row_smem[i] * rrms * norm_w[i]);
+}
+
 // ------------------------------------------------------------------ launchers
 int moe_route(int* ids, float* weights, const float* logits, int tokens, int E, int top, int softmax, int groups, int keep,
-              int renorm, void* stream) {
+              int renorm, const float* correction, float scale, void* stream) {
   PTL_REQUIRE(tokens >= 0 && E >= 1 && E <= kMoeMaxExperts && top >= 1 && top <= E, "moe_route: %d experts, top %d (at most %d experts)", E, top, kMoeMaxExperts);
   PTL_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
               "moe_route: %d experts in %d groups, %d kept, top %d", E, groups, keep, top);
+  PTL_REQUIRE(!correction || groups == 1, "moe_route: the correction goes with no groups");
   if (tokens == 0) return 0;
   return launch_kernel("moe_route", moe_route_kernel, dim3((tokens + 3) / 4), dim3(128), 0, as_stream(stream), ids, weights, logits,
-                       tokens, E, top, softmax, groups, keep, renorm);
+                       tokens, E, top, softmax, groups, keep, renorm, correction, scale);
 }
 
 int moe_plan(int* pos, int* tiles, int* meta, const int* ids, int n, int E, int max_tiles, int* wide, int max_wide, void* stream) {
@@ -691,7 +822,7 @@ int moe_gather(void* sorted, const void* x, const int* pos, const float* weights
 
 template <typename T>
 int moe_grouped(void* C, int ldc, const void* A, const void* W, const int* tiles, const int* meta, int max_tiles, int N, int K,
-                int gated, int tensor_cores, void* stream) {
+                int gated, int tensor_cores, GluForm form, void* stream) {
   PTL_REQUIRE(max_tiles >= 0 && N > 0 && K > 0 && (!gated || N % 2 == 0), "moe_grouped: bad sizes N=%d K=%d", N, K);
   if (max_tiles == 0) return 0;
   const int half = N / 2;
@@ -704,18 +835,18 @@ int moe_grouped(void* C, int ldc, const void* A, const void* W, const int* tiles
       if (gated) {
         if (int rc = raise_shared_memory("moe_grouped_mma", moe_grouped_mma_kernel<T, true>, kMmaSmem, raised_gated)) return rc;
         return launch_kernel("moe_grouped_mma", moe_grouped_mma_kernel<T, true>, grid, dim3(128), kMmaSmem, as_stream(stream),
-                             (T*)C, ldc, (const T*)A, (const T*)W, tiles, meta, N, K, stride, half);
+                             (T*)C, ldc, (const T*)A, (const T*)W, tiles, meta, N, K, stride, half, form);
       }
       if (int rc = raise_shared_memory("moe_grouped_mma", moe_grouped_mma_kernel<float, false>, kMmaSmem, raised_plain)) return rc;
       return launch_kernel("moe_grouped_mma", moe_grouped_mma_kernel<float, false>, grid, dim3(128), kMmaSmem, as_stream(stream),
-                           (float*)C, ldc, (const T*)A, (const T*)W, tiles, meta, N, K, stride, half);
+                           (float*)C, ldc, (const T*)A, (const T*)W, tiles, meta, N, K, stride, half, form);
     }
   }
   if (gated)
     return launch_kernel("moe_grouped", moe_grouped_kernel<T, T, true>, grid, dim3(256), 0, as_stream(stream), (T*)C, ldc, (const T*)A,
-                         (const T*)W, tiles, meta, N, K, stride, half);
+                         (const T*)W, tiles, meta, N, K, stride, half, form);
   return launch_kernel("moe_grouped", moe_grouped_kernel<T, float, false>, grid, dim3(256), 0, as_stream(stream), (float*)C, ldc,
-                       (const T*)A, (const T*)W, tiles, meta, N, K, stride, half);
+                       (const T*)A, (const T*)W, tiles, meta, N, K, stride, half, form);
 }
 
 template <typename T>
@@ -728,12 +859,29 @@ int moe_combine(float* out, const float* C, const void* shared_out, const int* p
                        (const T*)shared_out, pos, weights, top, width, scale_input, vec_ok);
 }
 
+template <typename T>
+int moe_combine_norm(float* residual, void* y, const float* C, const void* x, const void* add, const void* shared_out, const int* pos,
+                     const float* weights, const float* norm_w, int tokens, int top, int width, float eps, void* stream) {
+  PTL_REQUIRE(tokens >= 0 && top >= 1 && width > 0, "moe_combine_norm: bad sizes");
+  PTL_REQUIRE(residual && C && x && pos && weights && (!norm_w || (y && eps > 0.f)), "moe_combine_norm: missing operands");
+  if (tokens == 0) return 0;
+  const size_t smem = norm_w ? (size_t)width * sizeof(float) : 0;
+  PTL_REQUIRE(smem <= 200 * 1024, "moe_combine_norm: rows of %d do not fit the row buffer (max %d)", width, 200 * 1024 / 4);
+  static SmemRaised raised = {};
+  if (smem > 47 * 1024)
+    if (int rc = raise_shared_memory("moe_combine_norm", moe_combine_norm_kernel<T>, 200 * 1024, raised)) return rc;
+  const int vec_ok = width % 4 == 0 && aligned16(residual) && aligned16(C) && aligned16(x) && (!add || aligned16(add)) &&
+                     (!shared_out || aligned16(shared_out)) && (!norm_w || (aligned16(norm_w) && aligned16(y)));
+  return launch_kernel("moe_combine_norm", moe_combine_norm_kernel<T>, dim3(tokens), dim3(256), smem, as_stream(stream), residual, (T*)y,
+                       C, (const T*)x, (const T*)add, (const T*)shared_out, pos, weights, norm_w, top, width, eps, vec_ok);
+}
+
 }  // namespace ptl
 
 PTL_EXPORT int ptl_moe_tile_rows() { return ptl::kMoeTile; }
 PTL_EXPORT int ptl_moe_route(int* ids, float* weights, const float* logits, int tokens, int E, int top, int softmax, int groups,
-                             int keep, int renorm, void* stream) {
-  return ptl::moe_route(ids, weights, logits, tokens, E, top, softmax, groups, keep, renorm, stream);
+                             int keep, int renorm, const float* correction, float scale, void* stream) {
+  return ptl::moe_route(ids, weights, logits, tokens, E, top, softmax, groups, keep, renorm, correction, scale, stream);
 }
 PTL_EXPORT int ptl_moe_wide_rows() { return ptl::kMoeWide; }
 PTL_EXPORT int ptl_moe_plan(int* pos, int* tiles, int* meta, const int* ids, int n, int E, int max_tiles, int* wide, int max_wide,
@@ -742,8 +890,8 @@ PTL_EXPORT int ptl_moe_plan(int* pos, int* tiles, int* meta, const int* ids, int
 }
 // The grouped product over the wide tiles (bfloat16, tensor cores); -2 where the sizes are not taken.
 PTL_EXPORT int ptl_moe_grouped_wide_bf16(void* C, int ldc, const void* A, const void* W, const int* wide, const int* meta,
-                                         int max_wide, int N, int K, int gated, void* stream) {
-  return ptl::moe_grouped_wide(C, ldc, A, W, wide, meta, max_wide, N, K, gated, stream);
+                                         int max_wide, int N, int K, int gated, float limit, float alpha, float shift, void* stream) {
+  return ptl::moe_grouped_wide(C, ldc, A, W, wide, meta, max_wide, N, K, gated, ptl::GluForm{limit, alpha, shift}, stream);
 }
 #define PTL_MOE(SUFFIX, TYPE)                                                                                                     \
   PTL_EXPORT int ptl_moe_gather##SUFFIX(void* sorted, const void* x, const int* pos, const float* weights, int n, int top,         \
@@ -751,8 +899,15 @@ PTL_EXPORT int ptl_moe_grouped_wide_bf16(void* C, int ldc, const void* A, const 
     return ptl::moe_gather<TYPE>(sorted, x, pos, weights, n, top, width, scale_input, stream);                                    \
   }                                                                                                                               \
   PTL_EXPORT int ptl_moe_grouped##SUFFIX(void* C, int ldc, const void* A, const void* W, const int* tiles, const int* meta,        \
-                                         int max_tiles, int N, int K, int gated, int tensor_cores, void* stream) {                \
-    return ptl::moe_grouped<TYPE>(C, ldc, A, W, tiles, meta, max_tiles, N, K, gated, tensor_cores, stream);                       \
+                                         int max_tiles, int N, int K, int gated, int tensor_cores, float limit, float alpha,      \
+                                         float shift, void* stream) {                                                             \
+    return ptl::moe_grouped<TYPE>(C, ldc, A, W, tiles, meta, max_tiles, N, K, gated, tensor_cores,                                \
+                                  ptl::GluForm{limit, alpha, shift}, stream);                                                     \
+  }                                                                                                                               \
+  PTL_EXPORT int ptl_moe_combine_norm##SUFFIX(float* residual, void* y, const float* C, const void* x, const void* add,            \
+                                              const void* shared_out, const int* pos, const float* weights, const float* norm_w,  \
+                                              int tokens, int top, int width, float eps, void* stream) {                          \
+    return ptl::moe_combine_norm<TYPE>(residual, y, C, x, add, shared_out, pos, weights, norm_w, tokens, top, width, eps, stream); \
   }                                                                                                                               \
   PTL_EXPORT int ptl_moe_combine##SUFFIX(float* out, const float* C, const void* shared_out, const int* pos,                       \
                                          const float* weights, int tokens, int top, int width, int scale_input, void* stream) {   \

@@ -1,5 +1,5 @@
 // Row-wise kernels on the float32 residual stream and around it: the scaled embedding with a
-// sinusoidal position vector, the tanh cap of the logits, the clamped gated activation of a
+// sinusoidal position vector or with a row looked up by a pair of tokens, the tanh cap of the logits, the clamped gated activation of a
 // feed-forward, and the token-indexed side term of a layer.  All arithmetic is float32 (the
 // position angles float64); T is the element type of projections' results and of weights.
 #include "common.cuh"
@@ -32,6 +32,69 @@ __global__ void embed_scaled_kernel(float* __restrict__ out, const T* __restrict
     out[(size_t)t * width + i] = (bad ? 0.f : to_f32(src[i]) * scale) + a;
     if (i + 1 < width) out[(size_t)t * width + i + 1] = (bad ? 0.f : to_f32(src[i + 1]) * scale) + b;
   }
+}
+
+// out[t, :] = table[ids[t], :] * scale + pairs[row, :] with row = (ids before t * mul_prev + ids[t] * mul_cur) mod buckets,
+// and row = buckets for the token at position 0.  The token before a portion's first lies in `last` [slots], the
+// request's state: the block of that first token, and no other, reads it and puts the portion's last token in its
+// place.  Token rows of no request (tok_req < 0) give zeros.
+template <typename T>
+__global__ void __launch_bounds__(128)
+embed_bigram_kernel(float* __restrict__ out, const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ ids,
+                    const int* __restrict__ tok_req, const int* __restrict__ positions, const int* __restrict__ q_start,
+                    const int* __restrict__ state_slot, int* __restrict__ last, int num_slots, int width, int vocab, float scale,
+                    long long buckets, long long mul_prev, long long mul_cur, int vec_ok, int* __restrict__ status) {
+  __shared__ long long s_row;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int id = ids[t], r = tok_req[t];
+  const bool bad = id < 0 || id >= vocab;
+  if (threadIdx.x == 0) {
+    long long row = -1;
+    if (r >= 0) {
+      if (bad && status) atomicExch(status, 1);
+      row = buckets;
+      const int q0 = q_start[r];
+      int before = -1;
+      if (t == q0) {
+        const int slot = state_slot[r];
+        if (slot >= 0 && slot < num_slots) {
+          before = last[slot];
+          last[slot] = ids[q_start[r + 1] - 1];
+        }
+      } else {
+        before = ids[t - 1];
+      }
+      if (positions[t] > 0) {
+        if (before < 0 || before >= vocab) before = 0;
+        row = ((long long)before * mul_prev + (long long)(bad ? 0 : id) * mul_cur) % buckets;
+        if (row < 0) row += buckets;
+      }
+    }
+    s_row = row;
+  }
+  __syncthreads();
+  const long long row = s_row;
+  float* dst = out + (size_t)t * width;
+  if (row < 0 || bad) {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = 0.f;
+    return;
+  }
+  const T* a = table + (size_t)id * width;
+  const T* b = pairs + (size_t)row * width;
+  constexpr int VN = Vec16<T>::N;
+  if (vec_ok) {
+    for (int i = threadIdx.x * VN; i < width; i += blockDim.x * VN) {
+      const Vec16<T> va = load16(a + i), vb = load16(b + i);
+#pragma unroll
+      for (int e = 0; e < VN; e += 4)
+        *reinterpret_cast<float4*>(dst + i + e) = make_float4(fmaf(va.get(e), scale, vb.get(e)), fmaf(va.get(e + 1), scale, vb.get(e + 1)),
+                                                              fmaf(va.get(e + 2), scale, vb.get(e + 2)), fmaf(va.get(e + 3), scale, vb.get(e + 3)));
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = fmaf(to_f32(a[i]), scale, to_f32(b[i]));
 }
 
 __global__ void softcap_kernel(float* __restrict__ x, size_t n, float cap) {
@@ -189,6 +252,20 @@ int embed_scaled(float* out, const void* table, const int* ids, const int* posit
 }
 
 template <typename T>
+int embed_bigram(float* out, const void* table, const void* pairs, const int* ids, const int* tok_req, const int* positions,
+                 const int* q_start, const int* state_slot, int* last, int num_slots, int tokens, int width, int vocab, float scale,
+                 long long buckets, long long mul_prev, long long mul_cur, int* status, void* stream) {
+  PTL_REQUIRE(tokens >= 0 && width > 0 && vocab > 0 && buckets > 0 && num_slots > 0, "embed_bigram: bad sizes tokens=%d width=%d vocab=%d", tokens,
+              width, vocab);
+  PTL_REQUIRE(ids && tok_req && positions && q_start && state_slot && last, "embed_bigram: needs the step's integers and the last tokens' state");
+  if (tokens == 0) return 0;
+  const int vec_ok = width % Vec16<T>::N == 0 && aligned16(out) && aligned16(table) && aligned16(pairs);
+  return launch_kernel("embed_bigram", embed_bigram_kernel<T>, dim3(tokens), dim3(128), 0, as_stream(stream), out, (const T*)table,
+                       (const T*)pairs, ids, tok_req, positions, q_start, state_slot, last, num_slots, width, vocab, scale, buckets,
+                       mul_prev, mul_cur, vec_ok, status);
+}
+
+template <typename T>
 int clamped_glu(void* out, const void* gu, const float* bias, int tokens, int inter, float limit, float alpha, float up_shift,
                 void* stream) {
   PTL_REQUIRE(tokens >= 0 && inter > 0 && limit > 0.f, "clamped_glu: bad sizes tokens=%d inter=%d limit=%f", tokens, inter, limit);
@@ -243,6 +320,13 @@ PTL_EXPORT int ptl_softcap(float* x, long long n, float cap, void* stream) {
   PTL_EXPORT int ptl_embed_scaled##SUFFIX(float* out, const void* table, const int* ids, const int* positions, const double* freq, \
                                           int tokens, int width, int vocab, float scale, int* status, void* stream) {             \
     return ptl::embed_scaled<TYPE>(out, table, ids, positions, freq, tokens, width, vocab, scale, status, stream);                \
+  }                                                                                                                               \
+  PTL_EXPORT int ptl_embed_bigram##SUFFIX(float* out, const void* table, const void* pairs, const int* ids, const int* tok_req,     \
+                                          const int* positions, const int* q_start, const int* state_slot, int* last,             \
+                                          int num_slots, int tokens, int width, int vocab, float scale, long long buckets,        \
+                                          long long mul_prev, long long mul_cur, int* status, void* stream) {                     \
+    return ptl::embed_bigram<TYPE>(out, table, pairs, ids, tok_req, positions, q_start, state_slot, last, num_slots, tokens,      \
+                                   width, vocab, scale, buckets, mul_prev, mul_cur, status, stream);                              \
   }                                                                                                                               \
   PTL_EXPORT int ptl_clamped_glu##SUFFIX(void* out, const void* gu, const float* bias, int tokens, int inter, float limit,         \
                                          float alpha, float up_shift, void* stream) {                                             \

@@ -19,7 +19,8 @@
 // (see attention_simt.cu).  The list may be split over blockIdx.z and merged by a second kernel.
 // The kernel works `tokens` rows, or the rows that `items` names (the single tokens of a step
 // whose longer portions another kernel takes); partial results are indexed by the row itself.
-// Options: `sink` adds one term of score 0 (and no value) to the softmax's denominator; `temp_coef` != 0
+// Options: `sink` adds one term (and no value) to the softmax's denominator, of score 0 or, with `sink_logits` [H], of
+// that score for the head (not scaled); `temp_coef` != 0
 // multiplies the scores of the query at position p by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1);
 // `shared_v`: pages hold keys only and the value of a key is its first dv entries.  `bias_exp` = c > 0: head h takes
 // 2^(-c (h + 1) / H) * (p - j) off the score of key j.  `gate_col` >= 0: the result of head h is multiplied by the
@@ -430,7 +431,8 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
                         int bt_stride, int H, int G, int d, int dv, int page_size, float scale, int window, int keep,
                         int splits, int num_pages, int vec_ok, const int* __restrict__ items, int wide_ok, int shared_v,
                         int sink, float temp_coef, int temp_every, float bias_exp, int gate_col, int pool,
-                        const T* __restrict__ summary, const int* __restrict__ sum_bt, int sum_bt_stride, int sum_pages) {
+                        const T* __restrict__ summary, const int* __restrict__ sum_bt, int sum_bt_stride, int sum_pages,
+                        const float* __restrict__ sink_logits) {
   constexpr int kWaMaxPerLane = MPL;   // values of a head that a lane holds
   extern __shared__ float qs_all[];  // [warps][d]
   __shared__ float s_pr[kWaWarps][32];
@@ -603,10 +605,11 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
     for (int i = 0; i < kWaMaxPerLane; ++i) acc[i] = __fadd_rn(acc[i], acc_lo[i]);
   }
   if (splits == 1) {
-    if (sink) {            // the term of score 0 joins as a key would: the maximum may move to 0, and exp(0 - maximum) is added
-      const float m_all = fmaxf(m, 0.f);
+    if (sink) {            // the term joins as a key would: the maximum may move to its score z, and exp(z - maximum) is added
+      const float z = sink_logits ? sink_logits[h] : 0.f;
+      const float m_all = fmaxf(m, z);
       const float a = expf(m - m_all);
-      l = fmaf(l, a, expf(-m_all));
+      l = fmaf(l, a, expf(z - m_all));
 #pragma unroll
       for (int i = 0; i < kWaMaxPerLane; ++i) acc[i] *= a;
     }
@@ -639,7 +642,7 @@ template <typename T, int MPL>
 __global__ void __launch_bounds__(kWaWarps * 32)
 window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                               int out_stride, int H, int dv, int splits, int tokens, const int* __restrict__ items, int sink,
-                              const T* __restrict__ q, int q_stride, int gate_col) {
+                              const T* __restrict__ q, int q_stride, int gate_col, const float* __restrict__ sink_logits) {
   constexpr int kWaMaxPerLane = MPL;
   pdl_wait();
   pdl_launch_dependents();
@@ -654,7 +657,8 @@ window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ par
   float M = -INFINITY;
   for (int z = lane; z < splits; z += 32) M = fmaxf(M, part_ml[(idx0 + z) * 2]);
   M = warp_max(M);
-  if (sink) M = fmaxf(M, 0.f);
+  const float z_sink = sink_logits ? sink_logits[h] : 0.f;
+  if (sink) M = fmaxf(M, z_sink);
   float L = 0.f;
   float acc[kWaMaxPerLane];
 #pragma unroll
@@ -695,7 +699,7 @@ window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ par
     }
   }
   L = warp_sum(L);
-  if (sink) L += expf(-M);
+  if (sink) L += expf(z_sink - M);
   const float inv = L > 0.f ? 1.0f / L : 0.f;
   T* o = out + (size_t)t * out_stride + (size_t)h * dv;
   const T* gate = gate_col >= 0 ? q + (size_t)t * q_stride + gate_col + (size_t)h * dv : nullptr;
@@ -716,8 +720,9 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                      int bt_stride, int H, int G, int d, int dv, int page_size, float scale, int window, int keep, int splits,
                      int num_pages, const int* items, int shared_v, int sink, float temp_coef, int temp_every, float bias_exp,
                      int gate_col, int pool, const void* summary, const int* sum_bt, int sum_bt_stride, int sum_pages,
-                     void* stream) {
+                     const float* sink_logits, void* stream) {
   PTL_REQUIRE(tokens >= 0 && H > 0 && G > 0 && page_size > 0 && d > 0, "window_attention: bad sizes");
+  if (sink_logits) sink = 1;
   PTL_REQUIRE(pool == 0 || (summary && sum_bt && sum_pages > 0 && window > 0 && keep == 0 && !shared_v && !sink),
               "window_attention: means of blocks need their pages and a window, and go with no kept positions, shared values or sink");
   PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || gate_col + H * dv <= q_stride), "window_attention: bad bias or gate column");
@@ -748,12 +753,12 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                            as_stream(stream), (T*)out, part_acc, part_ml, (const T*)q, (const T*)cache, block_table, tok_req,      \
                            positions, q_stride, out_stride, bt_stride, H, G, d, dv, page_size, scale, window, keep, splits,        \
                            num_pages, vec_ok, items, wide_ok, shared_v, sink, temp_coef, temp_every, bias_exp, gate_col, pool,     \
-                           (const T*)summary, sum_bt, sum_bt_stride, sum_pages);                                                  \
+                           (const T*)summary, sum_bt, sum_bt_stride, sum_pages, sink_logits);                                     \
     if (rc || splits <= 1) return rc;                                                                                              \
     return launch_kernel("window_attention_merge", window_attention_merge_kernel<T, MPL>,                                          \
                          dim3((unsigned)((pairs + kWaWarps - 1) / kWaWarps)), dim3(kWaWarps * 32), 0, as_stream(stream), (T*)out,  \
                          (const float*)part_acc, (const float*)part_ml, out_stride, H, dv, splits, tokens, items, sink,            \
-                         (const T*)q, q_stride, gate_col);                                                                         \
+                         (const T*)q, q_stride, gate_col, sink_logits);                                                            \
   }
   if (dv <= 32 * 8) PTL_WA_LAUNCH(8)      // (value heads up to 256 keep the registers of 8 values per lane)
   PTL_WA_LAUNCH(16)
@@ -776,11 +781,11 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                                               int page_size, float scale, int window, int keep, int splits, int num_pages,         \
                                               const int* items, int shared_v, int sink, float temp_coef, int temp_every,           \
                                               float bias_exp, int gate_col, int pool, const void* summary, const int* sum_bt,      \
-                                              int sum_bt_stride, int sum_pages, void* stream) {                                    \
+                                              int sum_bt_stride, int sum_pages, const float* sink_logits, void* stream) {          \
     return ptl::window_attention<TYPE>(out, q, cache, block_table, tok_req, positions, part_acc, part_ml, tokens, q_stride,        \
                                        out_stride, bt_stride, H, G, d, dv, page_size, scale, window, keep, splits, num_pages,      \
                                        items, shared_v, sink, temp_coef, temp_every, bias_exp, gate_col, pool, summary, sum_bt,    \
-                                       sum_bt_stride, sum_pages, stream);                                                          \
+                                       sum_bt_stride, sum_pages, sink_logits, stream);                                             \
   }                                                                                                                                \
   PTL_EXPORT int ptl_head_norm_rotate_store##SUFFIX(void* proj, int tokens, int ld, int H, int G, int d, int dv, const float* wq,   \
                                                     const float* wk, float eps, const int* positions, const void* inv_freq,        \

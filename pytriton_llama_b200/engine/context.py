@@ -32,7 +32,7 @@ class LayerCacheView:
                                     # size [pages, kv_heads * page_size * (head_dim + value_dim)], keys first
     state: Optional[torch.Tensor]   # [slots, *state_shape] per-request state of this entry
     write: bool = True              # False: read what another run of a layer stored
-    states: Dict[str, torch.Tensor] = field(default_factory=dict)   # named per-request states: [slots, *shape] float32
+    states: Dict[str, torch.Tensor] = field(default_factory=dict)   # named per-request states: [slots, *shape], float32 unless the need says otherwise
     summary_group: Optional[GroupStepView] = None   # paging data of the entry's block means (``CacheNeed.pool_block``): the slot
                                                     # of a token is where the mean of the block it completes goes (-1: it completes none)
     summary: Optional[torch.Tensor] = None          # [pages, kv_heads * page_size * (head_dim + value_dim)], mean keys first

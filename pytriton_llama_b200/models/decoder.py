@@ -22,6 +22,8 @@ def _walk(part: Part, spec, prefix: str = ""):
 
 
 class DecoderModel:
+    EMBEDDING_ENTRY = -1     # the cache entry that holds the per-request states of the embedding part
+
     def __init__(self, spec: ModelSpec, runtime: Runtime):
         spec.validate()
         self.spec = spec
@@ -29,6 +31,7 @@ class DecoderModel:
         self.blocks = [build_part("block", b, runtime) for b in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm, runtime)
         self.embedding_norm = build_part("norm", spec.embedding_norm, runtime) if spec.embedding_norm is not None else None
+        self.embedding_part = build_part("embedding", spec.embedding_part, runtime) if spec.embedding_part is not None else None
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
 
@@ -36,6 +39,8 @@ class DecoderModel:
         roots = [(b, s) for b, s in zip(self.blocks, self.spec.layers)] + [(self.final_norm, self.spec.final_norm)]
         if self.embedding_norm is not None:
             roots.append((self.embedding_norm, self.spec.embedding_norm))
+        if self.embedding_part is not None:
+            roots.append((self.embedding_part, self.spec.embedding_part))
         return roots
 
     def any_part(self, predicate) -> bool:
@@ -92,6 +97,8 @@ class DecoderModel:
                     raise ValueError(f"cache entry {e.cache} is used by layers with different needs") from None
                 out[e.cache] = need
             out.setdefault(e.cache, need)
+        if self.embedding_part is not None:
+            out[self.EMBEDDING_ENTRY] = self.embedding_part.cache_need()
         return out
 
     # ------------------------------------------------------------------ forward
@@ -103,7 +110,12 @@ class DecoderModel:
         if begin is not None:
             begin()             # (what an operator set keeps per step, such as rotary angles, starts afresh)
         ctx.tokens = token_ids
-        if self.spec.position_vector is not None or self.spec.embedding_scale != 1.0:
+        if self.embedding_part is not None:
+            if self.spec.position_vector is not None or self.embedding_norm is not None:
+                raise ValueError("an embedding part goes with neither a position vector nor an embedding norm")
+            x, residual = None, self.embedding_part.start_stream(token_ids, self.embedding, self.spec.embedding_scale, ctx,
+                                                                 cache_views(self.EMBEDDING_ENTRY, True))
+        elif self.spec.position_vector is not None or self.spec.embedding_scale != 1.0:
             # scaled rows plus the position vector, in float32: this is the stream itself, nothing is left to add
             if self.spec.position_vector not in (None, "sinusoidal"):
                 raise ValueError(f"unknown position vector {self.spec.position_vector!r}")

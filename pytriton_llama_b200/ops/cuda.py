@@ -26,10 +26,12 @@ _ptr = ctypes.c_void_p
 _SIGNATURES = {
     "ptl_embed_gather": [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr],
     "ptl_add_rmsnorm": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr],
-    "ptl_silu_mul": [_ptr, _ptr, _c_int, _c_int, _ptr],
+    "ptl_gated_act": [_ptr, _c_int, _ptr, _c_int, _c_int, _c_int, _ptr],
     "ptl_rope_kv_write": [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ll, _ptr],
     "ptl_add_bias_rmsnorm": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr],
     "ptl_embed_scaled": [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_f, _ptr, _ptr],
+    "ptl_embed_bigram": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _c_ll, _c_ll, _c_ll,
+                         _ptr, _ptr],
     "ptl_clamped_glu": [_ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _c_f, _c_f, _ptr],
     "ptl_token_side": [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr],
     "ptl_causal_conv": [_ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int,
@@ -49,7 +51,9 @@ _SIGNATURES = {
                                  _ptr, _c_int, _c_ll, _ptr],
     "ptl_window_attention": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                              _c_int, _c_int, _c_f, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _c_int, _c_f, _c_int, _c_f, _c_int,
-                             _c_int, _ptr, _ptr, _c_int, _c_int, _ptr],
+                             _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr],
+    "ptl_pair_rotate_store": [_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr, _c_int, _c_ll,
+                              _ptr],
     "ptl_head_norm_rotate_store": [_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _c_f, _ptr, _ptr, _c_int, _c_int,
                                    _ptr, _ptr, _c_int, _c_ll, _ptr],
     "ptl_pool_blocks": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ll, _ptr],
@@ -69,7 +73,8 @@ _SIGNATURES = {
     "ptl_gla_scan": [_ptr, _ptr, _c_int, _ptr, _ptr, _c_f, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr, _c_f,
                      _ptr],
     "ptl_moe_gather": [_ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr],
-    "ptl_moe_grouped": [_ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr],
+    "ptl_moe_grouped": [_ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _ptr],
+    "ptl_moe_combine_norm": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_f, _ptr],
     "ptl_moe_combine": [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr],
     "ptl_paged_attention_simt": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int,
                                  _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_int, _ptr],
@@ -97,6 +102,15 @@ class NormedActivation:
     def materialise(self) -> torch.Tensor:
         """The normed activation as a plain tensor (for consumers that cannot apply the scale)."""
         return self.ops.finish_norm(self)
+
+
+class ExpertRows:
+    """The outputs of a step's chosen experts, sorted by expert: ``y`` float32 [rows, width], ``pos`` the row of every
+    (token, choice) (-1: a choice without one), ``weights`` their weights, ``x`` the tokens' input."""
+    __slots__ = ("y", "pos", "weights", "x", "top", "held")
+
+    def __init__(self, y, pos, weights, x, top, held):
+        self.y, self.pos, self.weights, self.x, self.top, self.held = y, pos, weights, x, top, held
 
 
 class KernelError(RuntimeError):
@@ -168,18 +182,20 @@ def load_library() -> ctypes.CDLL:
     lib.ptl_softcap.restype = _c_int
     lib.ptl_prefill_attention_opts_bf16.argtypes = [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                                     _c_int, _c_int, _c_f, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_f, _c_int,
-                                                    _c_int, _ptr, _ptr, _c_int, _c_int, _ptr]
+                                                    _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr]
     lib.ptl_prefill_attention_opts_bf16.restype = _c_int
     lib.ptl_moe_tile_rows.argtypes = []
     lib.ptl_moe_tile_rows.restype = _c_int
-    lib.ptl_moe_route.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr]
+    lib.ptl_moe_route.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _c_f, _ptr]
     lib.ptl_moe_route.restype = _c_int
     lib.ptl_moe_plan.argtypes = [_ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr]
     lib.ptl_moe_plan.restype = _c_int
     lib.ptl_moe_wide_rows.argtypes = []
     lib.ptl_moe_wide_rows.restype = _c_int
-    lib.ptl_moe_grouped_wide_bf16.argtypes = [_ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr]
+    lib.ptl_moe_grouped_wide_bf16.argtypes = [_ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _ptr]
     lib.ptl_moe_grouped_wide_bf16.restype = _c_int
+    lib.ptl_pair_angles.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr]
+    lib.ptl_pair_angles.restype = _c_int
     lib.ptl_lowrank_tanh_linear.argtypes = [_ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr]
     lib.ptl_lowrank_tanh_linear.restype = _c_int
     lib.ptl_head_linear_few_bf16.argtypes = _SIGNATURES["ptl_head_linear"]
@@ -276,16 +292,17 @@ class CudaOps:
 
     # ------------------------------------------------------------------ timing by class of kernels (diagnostic)
     KERNEL_CLASSES = {
-        "embed": "elementwise", "take_tokens": "elementwise", "silu_mul": "elementwise", "add_rmsnorm": "norm",
+        "embed": "elementwise", "take_tokens": "elementwise", "gated_act": "elementwise", "add_rmsnorm": "norm",
+        "embed_bigram": "elementwise", "_pair_angles": "rope", "pair_rotate_store": "rope",
         "embed_scaled": "elementwise", "softcap": "elementwise", "clamped_glu": "elementwise", "token_side": "token_input",
         "causal_conv": "recurrent", "selective_scan": "recurrent", "gated_delta_rule": "recurrent", "gated_head_norm": "norm",
         "kv_write_normed": "attention", "chunk_attention": "attention",
-        "linear": "product", "linear_add": "product", "gate_up_silu": "product", "gemm_tc": "product",
+        "linear": "product", "linear_add": "product", "gate_up_act": "product", "gemm_tc": "product",
         "_qkv_rope_product": "product", "rope_kv_write": "rope", "_rope_table": "rope",
         "paged_attention": "attention", "_attention_tensor_cores": "attention",
         "sample": "sampling", "token_logprobs": "sampling",
         "stream_mix_norm": "norm", "gelu_tanh": "elementwise", "qk_norm_rotate_store": "rope", "window_attention": "attention",
-        "gla_scan": "recurrent", "routed_experts": "experts",
+        "gla_scan": "recurrent", "routed_experts": "experts", "expert_rows": "experts", "combine_experts_add": "experts",
         "add_layernorm": "norm", "xielu": "elementwise", "lowrank_tanh_linear": "recurrent", "general_delta_scan": "recurrent",
         "latent_norm_store": "rope", "rotate_head_part": "rope", "head_linear": "product",
         "latent_gather": "attention", "causal_softmax_rows": "attention",
@@ -515,15 +532,23 @@ class CudaOps:
         return dtype == torch.bfloat16 and hidden % 8 == 0 and hidden >= 64
 
     def gate_up_silu(self, x, w_alternating: torch.Tensor) -> torch.Tensor:
-        out = self.gemm_tc(x, w_alternating, self.EPI_SILU_MUL)
-        if out is None and isinstance(x, NormedActivation):
-            out = self.gemm_tc(x.materialise(), w_alternating, self.EPI_SILU_MUL)
-        if out is None:
-            raise KernelError("gate_up_silu: sizes not taken; load the weights in the plain layout instead")
-        return out
+        return self.gate_up_act(x, w_alternating)
+
+    def gate_up_act(self, x, w_alternating: torch.Tensor, act: str = "silu", out: Optional[torch.Tensor] = None, column: int = 0) -> torch.Tensor:
+        """act(gate) * up of a product whose weight rows alternate gate_j, up_j, in its epilogue: [T, inter], or columns
+        ``column``.. of ``out``."""
+        epi = self.GATE_EPILOGUES[act]
+        kw = {} if out is None else dict(out=out, column=column)
+        y = self.gemm_tc(x, w_alternating, epi, **kw)
+        if y is None and isinstance(x, NormedActivation):
+            y = self.gemm_tc(x.materialise(), w_alternating, epi, **kw)
+        if y is None:
+            raise KernelError("gate_up_act: sizes not taken; load the weights in the plain layout instead")
+        return y
 
     # epilogues of the tensor-core product
-    EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SILU_MUL = 0, 1, 2, 3
+    EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SILU_MUL, EPI_GELU_MUL = 0, 1, 2, 3, 5
+    GATE_EPILOGUES = {"silu": EPI_SILU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
     def _tc_status_word(self):
         if getattr(self, "_tc_status", None) is None:
@@ -531,11 +556,11 @@ class CudaOps:
         return self._tc_status
 
     def gemm_tc(self, x, w: torch.Tensor, epi: int = 0, out: Optional[torch.Tensor] = None,
-                splits: int = 0, emit_norm=None):
+                splits: int = 0, emit_norm=None, column: int = 0):
         """x[M,K] @ w[N,K]^T in bfloat16 on the tcgen05 tensor cores with a fused epilogue.
         ``epi``: EPI_BF16 -> [M,N] bfloat16; EPI_F32 -> [M,N] float32; EPI_ADD_F32 adds into ``out``
-        (float32 [M,N], in place); EPI_SILU_MUL -> [M,N/2] bfloat16 for weights whose rows alternate
-        gate_j, up_j.  ``x`` may be a ``NormedActivation``: its row scale is applied before the
+        (float32 [M,N], in place); EPI_SILU_MUL, EPI_GELU_MUL -> [M,N/2] bfloat16 for weights whose rows alternate
+        gate_j, up_j (written to columns ``column``.. of ``out`` where that is given).  ``x`` may be a ``NormedActivation``: its row scale is applied before the
         epilogue.  ``emit_norm`` = (weight, eps) with EPI_ADD_F32 returns the ``NormedActivation`` of the
         norm that follows.  Returns None when the kernel does not take the sizes."""
         scale = None
@@ -554,9 +579,14 @@ class CudaOps:
                 raise KernelError("gemm_tc: the add epilogue needs the float32 tensor to add into")
             self._want(out, "out", torch.float32)
             ld = N
-        elif epi == self.EPI_SILU_MUL:
-            out = self.empty((M, N // 2), torch.bfloat16)
-            ld = N // 2
+        elif epi in (self.EPI_SILU_MUL, self.EPI_GELU_MUL):
+            if out is None:
+                out, column = self.empty((M, N // 2), torch.bfloat16), 0
+            else:
+                self._want(out, "out", torch.bfloat16)
+                if out.shape[0] != M or not 0 <= column <= out.shape[1] - N // 2 or column % 8:
+                    raise KernelError("gemm_tc: the columns of the result do not fit, or do not start at a multiple of 8")
+            ld = out.shape[1]
         elif epi == self.EPI_F32 and M > 64 and splits > 1:
             out = self.empty((splits, M, N), torch.float32)      # partial sums of the parts of the K range
             ld = N
@@ -581,7 +611,8 @@ class CudaOps:
             normed = NormedActivation(self.empty((M, N), torch.bfloat16), self.empty((M, width), torch.float32), 0,
                                       float(eps), weight, ops=self)
             slots = ctypes.c_int(0)
-        if M <= 8 and epi != self.EPI_SILU_MUL and splits == 0 and self.small_products:
+        out_ptr = out.data_ptr() + column * out.element_size()
+        if M <= 8 and epi not in (self.EPI_SILU_MUL, self.EPI_GELU_MUL) and splits == 0 and self.small_products:
             # a few tokens and a weight of a few megabytes (q|k|v and output projection of a decode step): the
             # product without tensor memory and clusters, whose latency is a third; -2 where it does not fit
             rc = self.lib.ptl_gemm_small_bf16(
@@ -598,14 +629,14 @@ class CudaOps:
                     return normed
                 return out
         if scale is None and emit_norm is None:
-            rc = self.lib.ptl_gemm_tc_bf16(_p(out), _p(x), _p(w), M, N, K, ld, epi, _p(self._tc_status_word()), splits,
+            rc = self.lib.ptl_gemm_tc_bf16(out_ptr, _p(x), _p(w), M, N, K, ld, epi, _p(self._tc_status_word()), splits,
                                            self._stream())
             if rc == -2:
                 return None
             self._check(rc)
             return out
         rc = self.lib.ptl_gemm_tc_bf16_norm(
-            _p(out), _p(x), _p(w), M, N, K, ld, epi, _p(self._tc_status_word()), splits,
+            out_ptr, _p(x), _p(w), M, N, K, ld, epi, _p(self._tc_status_word()), splits,
             _p(normed.xs) if normed else None, _p(normed.weight) if normed else None,
             _p(normed.sumsq) if normed else None, normed.sumsq.shape[1] if normed else 0,
             ctypes.byref(slots) if normed else None,
@@ -663,11 +694,25 @@ class CudaOps:
         return out
 
     def silu_mul(self, gu: torch.Tensor) -> torch.Tensor:
+        return self.gated_act(gu, "silu")
+
+    def gated_act(self, gu: torch.Tensor, act: str, out: Optional[torch.Tensor] = None, column: int = 0) -> torch.Tensor:
+        """gu [T, 2*inter] (gate columns first) -> act(gate) * up, [T, inter] or columns ``column``.. of ``out``; ``act``
+        "silu" or "gelu_tanh"."""
         self._want(gu, "gate_up")
+        if act not in ("silu", "gelu_tanh"):
+            raise KernelError(f"gated_act: activation {act!r}")
         tokens, two_i = gu.shape
-        out = self.empty((tokens, two_i // 2), gu.dtype)
-        fn = getattr(self.lib, "ptl_silu_mul" + _suffix(gu.dtype))
-        self._check(fn(_p(out), _p(gu), tokens, two_i // 2, self._stream()))
+        inter = two_i // 2
+        if out is None:
+            out, column = self.empty((tokens, inter), gu.dtype), 0
+        else:
+            self._want(out, "out", gu.dtype)
+            if out.shape[0] != tokens or not 0 <= column <= out.shape[1] - inter:
+                raise KernelError("gated_act: the columns of the result do not fit")
+        fn = getattr(self.lib, "ptl_gated_act" + _suffix(gu.dtype))
+        self._check(fn(out.data_ptr() + column * out.element_size(), out.shape[1], _p(gu), tokens, inter, int(act == "gelu_tanh"),
+                       self._stream()))
         return out
 
     def rope_kv_write(self, qkv: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[torch.Tensor],
@@ -753,6 +798,55 @@ class CudaOps:
         """Called by the model at the start of every forward pass: what was worked out for the last
         step's positions (the table of rotary angles) is forgotten."""
         self._rope_memo = None
+        self._pair_memo = {}
+
+    def _pair_angles(self, positions: torch.Tensor, freq: torch.Tensor, dims: int, amplitude: float) -> torch.Tensor:
+        """(cos, sin) [tokens, dims/2, 2] of position * freq, worked out once per forward pass for every table of
+        frequencies (float64) and used by every layer that has it."""
+        memo = getattr(self, "_pair_memo", None)
+        if memo is None:
+            memo = self._pair_memo = {}
+        key = (positions.data_ptr(), positions.shape[0], freq.data_ptr(), dims, float(amplitude))
+        have = memo.get(key)
+        if have is not None and have[0] == positions._version:
+            return have[1]
+        table = self.empty((positions.shape[0], dims // 2, 2), torch.float32)
+        self._check(self.lib.ptl_pair_angles(_p(table), _p(positions), _p(freq), positions.shape[0], dims // 2, float(amplitude),
+                                             self._stream()))
+        memo[key] = (positions._version, table, positions, freq)      # (held, so that their addresses are not given out again)
+        return table
+
+    def pair_rotate_store(self, proj: torch.Tensor, H: int, G: int, d: int, dv: int, bias: Optional[torch.Tensor],
+                          positions: torch.Tensor, freq: Optional[torch.Tensor], dims: int, amplitude: float,
+                          slots: Optional[torch.Tensor], cache: Optional[torch.Tensor], page_size: int,
+                          values_are_keys: bool = False) -> None:
+        """On proj [T, q | k (| v) | ...] (H heads of d, G of d, G of dv) + ``bias`` (float32, in the order of the columns):
+        the pairs (2i, 2i+1), i < dims/2, of every q and k head turned by position * freq[i] (float64 table; the angle
+        in 64 bits), cos and sin times ``amplitude``; q stays in place, k and v go to the tokens' slots of a cache whose
+        pages hold keys, then values.  ``values_are_keys``: proj has no v, the value is k before it is turned."""
+        self._want(proj, "proj")
+        self._want(positions, "positions", torch.int32)
+        if bias is not None:
+            self._want(bias, "bias", torch.float32)
+            if bias.numel() < (H + G) * d + (0 if values_are_keys else G * dv):
+                raise KernelError("pair_rotate_store: the bias is too short")
+        num_slots = 0
+        if G and cache is not None:
+            self._want(cache, "cache", proj.dtype)
+            self._want(slots, "slots", torch.int32)
+            if cache[0].numel() != G * page_size * (d + dv):
+                raise KernelError("pair_rotate_store: the cache's pages do not fit the heads")
+            num_slots = cache.shape[0] * page_size
+        table = None
+        if freq is not None and dims > 0:
+            self._want(freq, "freq", torch.float64)
+            if freq.numel() < dims // 2:
+                raise KernelError("pair_rotate_store: fewer frequencies than pairs")
+            table = self._pair_angles(positions, freq, dims, amplitude)
+        fn = getattr(self.lib, "ptl_pair_rotate_store" + _suffix(proj.dtype))
+        self._check(fn(_p(proj), proj.shape[0], proj.shape[1], H, G, d, dv, _p(bias), _p(table), int(dims) if table is not None else 0,
+                       int(bool(values_are_keys)), _p(slots) if num_slots else None, _p(cache) if num_slots else None, page_size,
+                       num_slots, self._stream()))
 
     def _rope_table(self, positions: torch.Tensor, inv_freq: torch.Tensor, half: int) -> torch.Tensor:
         """(cos, sin) [tokens, half] of this step's angles, worked out once per forward pass and used by every layer."""
@@ -895,6 +989,27 @@ class CudaOps:
         fn = getattr(self.lib, "ptl_embed_scaled" + _suffix(table.dtype))
         self._check(fn(_p(out), _p(table), _p(ids), _p(positions), _p(freq), ids.shape[0], width, table.shape[0], float(scale),
                        _p(self._status), self._stream()))
+        return out
+
+    def embed_bigram(self, ids: torch.Tensor, table: torch.Tensor, scale: float, pairs: torch.Tensor, mul_prev: int, mul_cur: int,
+                     ctx, last: torch.Tensor) -> torch.Tensor:
+        """float32 [T, width]: table[ids] * scale + pairs[row], row = (token before * mul_prev + token * mul_cur) mod buckets
+        for ``pairs`` [buckets + 1, width], its last row for a request's first token.  ``last`` int32 [slots, 1] holds each
+        request's last token and is moved on."""
+        self._want(ids, "ids", torch.int32)
+        self._want(table, "table")
+        self._want(pairs, "pair table", table.dtype)
+        self._want(last, "last tokens", torch.int32)
+        width = table.shape[1]
+        if pairs.shape[1] != width or pairs.shape[0] < 2:
+            raise KernelError("embed_bigram: the pair table does not fit")
+        for name in ("positions", "tok_req", "q_start", "state_slot"):
+            self._want(getattr(ctx, name), name, torch.int32)
+        out = self.empty((ids.shape[0], width), torch.float32)
+        fn = getattr(self.lib, "ptl_embed_bigram" + _suffix(table.dtype))
+        self._check(fn(_p(out), _p(table), _p(pairs), _p(ids), _p(ctx.tok_req), _p(ctx.positions), _p(ctx.q_start), _p(ctx.state_slot),
+                       _p(last), last.shape[0], ids.shape[0], width, table.shape[0], float(scale), pairs.shape[0] - 1, int(mul_prev),
+                       int(mul_cur), _p(self._status), self._stream()))
         return out
 
     def softcap(self, logits: torch.Tensor, cap: float) -> None:
@@ -1112,13 +1227,14 @@ class CudaOps:
 
     def window_attention(self, q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, tok_req: torch.Tensor,
                          positions: torch.Tensor, H: int, G: int, d: int, dv: int, page_size: int, scale: float, window: int = 0,
-                         keep_first: int = 0, splits: int = 1, hints=None, sink: bool = False, temp_coef: float = 0.0,
+                         keep_first: int = 0, splits: int = 1, hints=None, sink=False, temp_coef: float = 0.0,
                          temp_every: int = 1, shared_values: bool = False, distance_bias: float = 0.0, gate_column: int = -1,
                          pool: int = 0, summary: Optional[torch.Tensor] = None,
-                         summary_table: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         summary_table: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+                         column: int = 0) -> torch.Tensor:
         """Softmax attention of every token over the keys j <= p of its request with p - j < window or j < keep_first
-        (window 0: all); q is [T, >= H*d], the result [T, H*dv].  ``sink``: one more term of score 0 in the
-        denominator; ``temp_coef``: scores of the query at position p times 1 + temp_coef * ln(floor((p + 1) /
+        (window 0: all); q is [T, >= H*d], the result [T, H*dv], or columns ``column``.. of ``out``.  ``sink``: one more
+        term in the denominator, of score 0 (True) or of the head's own score (float32 [H]); ``temp_coef``: scores of the query at position p times 1 + temp_coef * ln(floor((p + 1) /
         temp_every) + 1); ``shared_values``: the cache's pages hold keys only and a key's first dv entries are its value.
         ``distance_bias`` = c: head h takes 2^(-c (h + 1) / H) * (p - j) off its scores; ``gate_column``: the heads are
         multiplied by the sigmoid of q's columns from there; ``pool`` = P with ``summary`` (pages of mean keys and
@@ -1131,7 +1247,19 @@ class CudaOps:
         if cache[0].numel() != G * page_size * (d + (0 if shared_values else dv)):
             raise KernelError("window_attention: the cache's pages do not fit the heads")
         tokens = q.shape[0]
-        out = self.empty((tokens, H * dv), q.dtype)
+        if out is None:
+            out, column = self.empty((tokens, H * dv), q.dtype), 0
+        else:
+            self._want(out, "out", q.dtype)
+            if out.shape[0] != tokens or not 0 <= column <= out.shape[1] - H * dv:
+                raise KernelError("window_attention: the columns of the result do not fit")
+        whole, out = out, out if not column else out[:, column:]          # (the kernels take the address and the row pitch)
+        sink_logits = None
+        if isinstance(sink, torch.Tensor):
+            self._want(sink, "sink", torch.float32)
+            if sink.numel() != H:
+                raise KernelError("window_attention: one sink score per head")
+            sink, sink_logits = True, sink
         if pool and window:
             self._want(summary, "summary", q.dtype)
             self._want(summary_table, "summary_table", torch.int32)
@@ -1141,19 +1269,20 @@ class CudaOps:
         else:
             pooled = (0, None, None, 0, 0)
         options = (int(bool(shared_values)), int(bool(sink)), float(temp_coef), int(temp_every), float(distance_bias),
-                   int(gate_column), *pooled)
-        if (q.dtype == torch.bfloat16 and d == dv and d in (64, 128) and not shared_values and self._work(hints, "prefill_tiles") is not None
+                   int(gate_column), *pooled, _p(sink_logits))
+        aligned = out.data_ptr() % 16 == 0 and out.stride(0) % 2 == 0
+        if (aligned and q.dtype == torch.bfloat16 and d == dv and d in (64, 128) and not shared_values and self._work(hints, "prefill_tiles") is not None
                 and self._work(hints, "decode_items") is not None and os.environ.get("PTL_WINDOW_TC", "1") != "0"):
             if self._window_attention_tensor_cores(out, q, cache, block_table, tok_req, positions, H, G, d, page_size, scale,
                                                    window, keep_first, hints, options):
-                return out
+                return whole
         longest = getattr(hints, "max_ctx_len", 0) or block_table.shape[1] * page_size
         if window:
             longest = min(longest, window + keep_first + (longest // pooled[0] + 32 if pooled[0] else 0))
         splits = self._window_splits(tokens, H, longest)
         self._window_attention_simt(out, q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window,
                                     keep_first, splits, None, options)
-        return out
+        return whole
 
     def _window_splits(self, tokens: int, H: int, longest: int) -> int:
         """Parts of a token's key list for the CUDA-core kernel: enough warps to fill the SMs, at least 64 keys each."""
@@ -1164,9 +1293,8 @@ class CudaOps:
                                keep_first, splits, rows, options=(0, 0, 0.0, 1)) -> None:
         """``rows``: None for every token row, else (int32 row indices or None for 0..n-1, n).  ``options``: (values
         inside the keys, sink term, temperature coefficient, temperature step[, distance bias exponent, gate column,
-        block length of the means, their pages, their block table, its width, number of their pages])."""
-        if len(options) == 4:
-            options = (*options, 0.0, -1, 0, None, None, 0, 0)
+        block length of the means, their pages, their block table, its width, number of their pages[, sink scores]])."""
+        options = (*options, *(0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0, None)[len(options):])
         tokens = q.shape[0]
         items, n_rows = (None, tokens) if rows is None else rows
         part_acc = part_ml = None
@@ -1175,19 +1303,19 @@ class CudaOps:
             part_ml = self.empty((tokens, H, splits, 2), torch.float32)
         fn = getattr(self.lib, "ptl_window_attention" + _suffix(q.dtype))
         self._check(fn(_p(out), _p(q), _p(cache), _p(block_table), _p(tok_req), _p(positions), _p(part_acc), _p(part_ml), n_rows,
-                       q.shape[1], out.shape[1], block_table.shape[1], H, G, d, dv, page_size, float(scale), int(window),
+                       q.shape[1], out.stride(0), block_table.shape[1], H, G, d, dv, page_size, float(scale), int(window),
                        int(keep_first), int(splits), cache.shape[0], _p(items), *options, self._stream()),
                     kernels=2 if splits > 1 else 1)
 
     def _window_attention_tensor_cores(self, out, q, cache, block_table, tok_req, positions, H, G, d, page_size, scale, window,
-                                       keep_first, hints, options=(0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0)) -> bool:
+                                       keep_first, hints, options=(0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0, None)) -> bool:
         """bfloat16, key and value heads of 64 or 128: the portions of a step on the tensor cores (the warp-level prompt
         kernel, which walks the kept first keys as key tiles of their own before the window's), its single tokens on
         the CUDA-core kernel with their key lists split; both write their rows of ``out``."""
         dec, tiles = hints.work["decode_items"], hints.work["prefill_tiles"]
         if tiles.items:
             rc = self.lib.ptl_prefill_attention_opts_bf16(
-                _p(out), _p(q), _p(cache), _p(block_table), _p(tiles.tensor), tiles.items, q.shape[1], H * d, block_table.shape[1],
+                _p(out), _p(q), _p(cache), _p(block_table), _p(tiles.tensor), tiles.items, q.shape[1], out.stride(0), block_table.shape[1],
                 H, G, d, page_size, float(scale), int(window), int(keep_first), cache.shape[0], *options[1:], self._stream())
             if rc == -2:
                 return False
@@ -1567,26 +1695,52 @@ class CudaOps:
     MOE_WIDE_MIN_ROWS = int(os.environ.get("PTL_MOE_WIDE_MIN", "512"))   # (token, choice) pairs from which tiles of 128 rows pay
 
     def routed_experts(self, x: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, top: int,
-                       scale_input: bool, shared: Optional[torch.Tensor], score: str = "sigmoid", groups: int = 1,
-                       keep_groups: int = 1, renormalise: bool = False) -> torch.Tensor:
+                       scale_input: bool, shared: Optional[torch.Tensor], **routing) -> torch.Tensor:
         """x [T, width], router logits float32 [T, E], expert weights [E, 2*inter, width] (gate rows, then up rows) and
         [E, width, inter]: every token's ``top`` experts by sigmoid(logit), weighted by that score on the expert's input
-        (``scale_input``) or output, summed, plus ``shared`` [T, width]; float32 [T, width].  ``score`` "softmax": the
-        scores are the softmax over all experts; ``groups`` > 1: only experts of the ``keep_groups`` groups of neighbours
-        with the largest best score can be chosen; ``renormalise``: chosen scores divided by their sum.  Six kernels and no word
+        (``scale_input``) or output, summed, plus ``shared`` [T, width]; float32 [T, width].  Six kernels and no word
         back to the host: route, plan (sort by expert), gather, two grouped products, combine.  The products walk tiles
-        of 32 rows of one expert; in bfloat16 steps with many tokens walk tiles of 128 rows."""
+        of 32 rows of one expert; in bfloat16 steps with many tokens walk tiles of 128 rows.  ``routing``: see ``expert_rows``."""
+        if shared is not None:
+            self._want(shared, "shared", x.dtype)
+        if logits.shape[1] != w_gate_up.shape[0]:
+            raise KernelError("routed_experts: experts without weights go with combine_experts_add")
+        rows = self.expert_rows(x, logits, w_gate_up, w_down, top, scale_input, **routing)
+        T, width = x.shape
+        out = self.empty((T, width), torch.float32)
+        self._check(getattr(self.lib, "ptl_moe_combine" + _suffix(x.dtype))(_p(out), _p(rows.y), _p(shared), _p(rows.pos), _p(rows.weights), T,
+                                                                            top, width, int(bool(scale_input)), self._stream()))
+        return out
+
+    def expert_rows(self, x: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, top: int,
+                    scale_input: bool = False, score: str = "sigmoid", groups: int = 1, keep_groups: int = 1,
+                    renormalise: bool = False, correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
+                    clamped: Optional[Tuple[float, float, float]] = None) -> "ExpertRows":
+        """Everything of ``routed_experts`` up to the experts' outputs, which lie sorted by expert.  ``score`` "softmax": the
+        scores are the softmax over all experts; ``groups`` > 1: only experts of the ``keep_groups`` groups of neighbours
+        with the largest best score can be chosen; ``correction`` float32 [E]: experts are chosen by score + correction and
+        weighted by the score; ``renormalise``: chosen scores divided by their sum; ``weight_scale`` multiplies the weights.
+        Logits beyond the experts that have weights belong to experts that hand their input on (they get no row).
+        ``clamped`` = (limit, alpha, shift): an expert's inner value is min(g, limit) * sigmoid(alpha * min(g, limit)) *
+        (clamp(u, +-limit) + shift) instead of silu(g) * u."""
         self._want(x, "x")
         self._want(logits, "logits", torch.float32)
         self._want(w_gate_up, "expert gate/up weights", x.dtype)
         self._want(w_down, "expert down weights", x.dtype)
-        if shared is not None:
-            self._want(shared, "shared", x.dtype)
         T, width = x.shape
         E, two_inter, _ = w_gate_up.shape
         inter = two_inter // 2
-        if logits.shape[1] != E or tuple(w_down.shape) != (E, width, inter) or w_gate_up.shape[2] != width:
-            raise KernelError("routed_experts: shapes do not fit")
+        E_all = logits.shape[1]
+        if E_all < E or tuple(w_down.shape) != (E, width, inter) or w_gate_up.shape[2] != width:
+            raise KernelError("expert_rows: shapes do not fit")
+        if E_all > E and scale_input:
+            raise KernelError("expert_rows: experts without weights go with weights on the output")
+        if correction is not None:
+            self._want(correction, "correction", torch.float32)
+            if correction.numel() != E_all:
+                raise KernelError("expert_rows: one correction per expert")
+        if score not in ("sigmoid", "softmax"):
+            raise KernelError(f"expert_rows: score {score!r}")
         n = T * top
         tile = self.lib.ptl_moe_tile_rows()
         max_tiles = -(-n // tile) + min(E, n)
@@ -1599,10 +1753,9 @@ class CudaOps:
         wide = ints[2 * n + 3 * max_tiles:2 * n + 3 * max_tiles + 3 * max_wide] if use_wide else None
         meta = ints[2 * n + 3 * max_tiles + 3 * max_wide:]
         weights = self.empty((n,), torch.float32)
-        if score not in ("sigmoid", "softmax"):
-            raise KernelError(f"routed_experts: score {score!r}")
-        self._check(self.lib.ptl_moe_route(_p(ids), _p(weights), _p(logits), T, E, top, int(score == "softmax"), int(groups),
-                                           int(keep_groups) if groups > 1 else 1, int(bool(renormalise)), stream))
+        self._check(self.lib.ptl_moe_route(_p(ids), _p(weights), _p(logits), T, E_all, top, int(score == "softmax"), int(groups),
+                                           int(keep_groups) if groups > 1 else 1, int(bool(renormalise)), _p(correction),
+                                           float(weight_scale), stream))
         self._check(self.lib.ptl_moe_plan(_p(pos), _p(tiles), _p(meta), _p(ids), n, E, max_tiles, _p(wide), max_wide, stream))
         rows = max_tiles * tile
         sorted_x = self.empty((rows, width), x.dtype)
@@ -1613,18 +1766,42 @@ class CudaOps:
         tc = int(self.moe_tensor_cores)
         grouped = getattr(self.lib, "ptl_moe_grouped" + sfx)
         y = self.empty((rows, width), torch.float32)
+        form = tuple(float(v) for v in clamped) if clamped is not None else (0.0, 0.0, 0.0)
         if use_wide:
             self._check(self.lib.ptl_moe_grouped_wide_bf16(_p(hidden), inter, _p(sorted_x), _p(w_gate_up), _p(wide), _p(meta), max_wide,
-                                                           two_inter, width, 1, stream))
+                                                           two_inter, width, 1, *form, stream))
             self._check(self.lib.ptl_moe_grouped_wide_bf16(_p(y), width, _p(hidden), _p(w_down), _p(wide), _p(meta), max_wide, width,
-                                                           inter, 0, stream))
+                                                           inter, 0, *form, stream))
         else:
-            self._check(grouped(_p(hidden), inter, _p(sorted_x), _p(w_gate_up), _p(tiles), _p(meta), max_tiles, two_inter, width, 1, tc, stream))
-            self._check(grouped(_p(y), width, _p(hidden), _p(w_down), _p(tiles), _p(meta), max_tiles, width, inter, 0, tc, stream))
-        out = self.empty((T, width), torch.float32)
-        self._check(getattr(self.lib, "ptl_moe_combine" + sfx)(_p(out), _p(y), _p(shared), _p(pos), _p(weights), T, top, width,
-                                                               int(bool(scale_input)), stream))
-        return out
+            self._check(grouped(_p(hidden), inter, _p(sorted_x), _p(w_gate_up), _p(tiles), _p(meta), max_tiles, two_inter, width, 1, tc, *form,
+                                stream))
+            self._check(grouped(_p(y), width, _p(hidden), _p(w_down), _p(tiles), _p(meta), max_tiles, width, inter, 0, tc, *form, stream))
+        return ExpertRows(y, pos, weights, x, top, (ints, sorted_x, hidden))
+
+    def combine_experts_add(self, rows: "ExpertRows", residual: torch.Tensor, add: Optional[torch.Tensor] = None,
+                            shared: Optional[torch.Tensor] = None, next_norm=None) -> Optional[torch.Tensor]:
+        """residual (float32 [T, width], in place) += ``add`` + ``shared`` + the weighted sum of the chosen experts' outputs,
+        the token's own input standing for a choice without a row.  ``next_norm`` = (weight, eps): returns the RMS norm
+        of the new residual in x's type as well.  One kernel."""
+        x = rows.x
+        T, width = x.shape
+        self._want(residual, "residual", torch.float32)
+        for name, t in (("add", add), ("shared", shared)):
+            if t is not None:
+                self._want(t, name, x.dtype)
+                if tuple(t.shape) != (T, width):
+                    raise KernelError(f"combine_experts_add: {name} does not fit")
+        if tuple(residual.shape) != (T, width):
+            raise KernelError("combine_experts_add: the residual does not fit")
+        y, weight, eps = None, None, 0.0
+        if next_norm is not None:
+            weight, eps = next_norm
+            self._want(weight, "norm weight", torch.float32)
+            y = self.empty((T, width), x.dtype)
+        fn = getattr(self.lib, "ptl_moe_combine_norm" + _suffix(x.dtype))
+        self._check(fn(_p(residual), _p(y), _p(rows.y), _p(x), _p(add), _p(shared), _p(rows.pos), _p(rows.weights), _p(weight), T, rows.top,
+                       width, float(eps), self._stream()))
+        return y
 
     def token_logprobs(self, logits: torch.Tensor, tokens: torch.Tensor) -> torch.Tensor:
         """log softmax(logits[row])[tokens[row]] as float32 [rows]."""

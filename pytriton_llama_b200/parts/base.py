@@ -1,9 +1,9 @@
 """Interfaces and registry of the parts a decoder layer is put together from.
 
-A part is one of six categories: ``mixer`` (attention, a selective scan, a delta rule, or several
+A part is one of seven categories: ``mixer`` (attention, a selective scan, a delta rule, or several
 side by side), ``ffn``, ``norm``, ``position``, ``token_input`` (a term that depends on the
-token itself, added to the stream inside a layer) and ``block`` (how the others are arranged
-around the residual stream).  A part is described
+token itself, added to the stream inside a layer), ``embedding`` (how the stream starts where that is
+more than a scaled row per token) and ``block`` (how the others are arranged around the residual stream).  A part is described
 by a ``PartSpec`` (kind + its sizes and constants + where its tensors are in the checkpoint) and
 built by ``build_part``; it never sees the model's configuration and does not know which model
 it is in.  New kinds are added with ``register_part`` from anywhere, tests included.
@@ -31,6 +31,8 @@ Contracts (``T`` = tokens of the step, all tensors on the runtime's device):
   the float32 ``residual`` in place;
 * a mixer or ffn with the class attribute ``fuses_residual = True`` is called with
   ``residual=<float32 [T, H]>`` as well and may add its output into it and return None;
+* embedding: ``cache_need() -> CacheNeed`` of kind "none" (its per-request states);
+  ``start_stream(token_ids, table, scale, ctx, cache) -> float32 [T, H]``;
 * block: ``forward(x, residual, ctx, cache) -> (x, residual)``.
 """
 from __future__ import annotations
@@ -40,7 +42,7 @@ from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
 
-CATEGORIES = ("mixer", "ffn", "norm", "position", "token_input", "block")
+CATEGORIES = ("mixer", "ffn", "norm", "position", "token_input", "embedding", "block")
 
 
 @dataclass(frozen=True)
@@ -68,8 +70,8 @@ class CacheNeed:
     (only the keys of the block of ``window`` positions, counted from position 0, that the next
     query lies in) or "none".  ``value_dim``: size of a value head where it differs from
     ``head_dim`` (0: the same).  ``state_shape``/``state_dtype``: per-request state of fixed size
-    (None if none).  ``states``: further per-request states by name, float32, as (name, shape)
-    pairs; a mixer made of several lists those of all its members.  ``keep_first`` (kind "window"):
+    (None if none).  ``states``: further per-request states by name, as (name, shape) pairs (float32) or
+    (name, shape, dtype) triples; a mixer made of several lists those of all its members.  ``keep_first`` (kind "window"):
     the keys of positions below it stay visible, and held, whatever the window has passed.
     ``shared_values``: a key's first ``value_dim`` entries are its value; no values are stored.
     ``pool_block`` = P > 0: beside its pages of keys and values the entry keeps, in pages of their own, one mean key
@@ -81,7 +83,7 @@ class CacheNeed:
     state_shape: Optional[Tuple[int, ...]] = None
     state_dtype: Optional[torch.dtype] = None
     value_dim: int = 0
-    states: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
+    states: Tuple[Tuple[Any, ...], ...] = ()
     keep_first: int = 0
     shared_values: bool = False
     pool_block: int = 0
@@ -146,6 +148,26 @@ def build_part(category: str, spec: PartSpec, runtime: Runtime):
     except KeyError:
         raise KeyError(f"no {category} part of kind {spec.kind!r}; registered: {part_kinds(category)}") from None
     return cls(spec, runtime)
+
+
+class NormedInput:
+    """The input of a norm's reader, made ahead of time by the kernel that completed the residual: ``y`` is the normed
+    activation of the norm whose weight is ``weight`` (what ``RMSNorm.forward`` passes through untouched)."""
+
+    def __init__(self, y: torch.Tensor, weight: torch.Tensor):
+        self.y, self.weight = y, weight
+
+    def materialise(self) -> torch.Tensor:
+        return self.y
+
+
+def side_stream(runtime: Runtime) -> "torch.cuda.Stream":
+    """One stream beside the launching one, shared by all parts of a model that run two things side by side."""
+    stream = getattr(runtime, "_side_stream", None)
+    if stream is None:
+        stream = torch.cuda.Stream(runtime.device)
+        setattr(runtime, "_side_stream", stream)
+    return stream
 
 
 class Part:

@@ -3,11 +3,16 @@
 lite_llama/models/llama.py:136-162: pre-norm block.  The stream is carried as two tensors: the
 output of the last sub-layer (not yet added) and the float32 residual; each norm first adds the
 former into the latter.  The block returns its feed-forward output un-added, so the next block's
-first norm (or the model's final norm, :219) folds it in.
+first norm (or the model's final norm, :219) folds it in.  ``SharedNormBlock`` is the arrangement with one
+norm whose output both sub-layers read.
 """
 from __future__ import annotations
 
-from .base import Part, PartSpec, Runtime, build_part, register_part
+import os
+
+import torch
+
+from .base import NormedInput, Part, PartSpec, Runtime, build_part, register_part, side_stream
 
 
 @register_part("block", "pre_norm")
@@ -65,3 +70,107 @@ class PreNormBlock(Part):
             if getattr(part, "emits_normed", False) and getattr(following_norm, "deferrable", False):
                 kw["next_norm"] = (following_norm.weight, following_norm.eps)
         return part.forward(y, *args, **kw)
+
+
+@register_part("block", "shared_norm")
+class SharedNormBlock(Part):
+    """One norm, both sub-layers on its output, both outputs added into the stream: with h = norm1(x),
+    x <- x + (mixer(h) + ffn(h)).
+
+    Nested parts: ``norm1``, ``mixer``, optionally ``ffn``.  The mixer has ``write_inner`` (its heads' outputs into columns
+    of a buffer), ``inner_width`` and ``w_o``.  A feed-forward with ``write_inner`` as well (a gated MLP) shares one output
+    product with the mixer: the inputs of both last projections lie side by side in one buffer, their weights side by side
+    in one matrix, and the product's sum over them is the layer's addition to the stream.  One with ``begin`` and
+    ``finish`` (routed experts) adds the mixer's output, its own and the next norm up in its last kernel.
+
+    On a CUDA device the two sub-layers run side by side in time: the feed-forward on a second stream that starts when
+    the normed input is ready and is joined before the sum.  ``PTL_PARALLEL_STREAMS=0`` runs them one after the other."""
+
+    takes_next_norm = True
+
+    def __init__(self, spec: PartSpec, runtime: Runtime):
+        super().__init__(spec, runtime)
+        self.norm1 = build_part("norm", spec.parts["norm1"], runtime)
+        self.mixer = build_part("mixer", spec.parts["mixer"], runtime)
+        self.ffn = build_part("ffn", spec.parts["ffn"], runtime) if "ffn" in spec.parts else None
+        self.routed = self.ffn is not None and hasattr(self.ffn, "begin")
+        if self.ffn is not None and not self.routed and not hasattr(self.ffn, "write_inner"):
+            raise ValueError(f"a feed-forward of kind {spec.parts['ffn'].kind!r} cannot stand beside a mixer")
+        if self.routed:
+            self.norm1.deferrable = False      # experts and router read the normed input itself, not a product's preparation of it
+        self.w_out = None
+        self.mixer_column, self.padded = 0, False
+
+    def children(self):
+        parts = {"norm1": self.norm1, "mixer": self.mixer, "ffn": self.ffn}
+        return {k: v for k, v in parts.items() if v is not None}
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def after_load(self) -> None:
+        self.w_out = self.mixer.w_o
+        if self.ffn is None or self.routed:
+            return
+        # the feed-forward's columns first; both parts start at multiples of 8 columns (with zeros between, in the buffer
+        # and in the weight), so that the kernels that write them keep their alignment
+        pad = lambda w: torch.nn.functional.pad(w, (0, -w.shape[1] % 8))
+        f, m = pad(self.ffn.w_down), pad(self.mixer.w_o)
+        self.padded = f.shape[1] != self.ffn.inner_width or m.shape[1] != self.mixer.inner_width
+        self.mixer_column = f.shape[1]
+        self.w_out = torch.cat([f, m], dim=1).contiguous()
+        self.ffn.w_down = self.mixer.w_o = None          # the joint weight is the one that is used
+
+    def forward(self, x, residual, ctx, cache, next_norm=None):
+        ops = self.rt.ops
+        y, residual = self.norm1.forward(x, residual)
+        prepared = y
+        if hasattr(y, "materialise") and (isinstance(y, NormedInput) or self.routed):
+            y = prepared = y.materialise()
+        T, dtype = prepared.shape[0], self.rt.dtype
+        width = self.mixer.inner_width
+        if self.ffn is None:
+            out = ops.empty((T, width), dtype)
+            self.mixer.write_inner(y, ctx, cache, out, 0, 1.0)
+            return self._add(out, self.w_out, residual, next_norm), residual
+        fork = self.rt.device.type == "cuda" and os.environ.get("PTL_PARALLEL_STREAMS", "1") != "0"
+        if self.routed:
+            begun = self._beside(fork, lambda: self.ffn.begin(y))
+            out = ops.empty((T, width), dtype)
+            self.mixer.write_inner(y, ctx, cache, out, 0, 1.0)
+            add = ops.linear_add(out, self.w_out, residual)            # None: already added
+            self._join(fork)
+            following = (next_norm.weight, next_norm.eps) if self._plain_rms(next_norm) else None
+            normed = self.ffn.finish(begun, residual, add=add, next_norm=following)
+            return (NormedInput(normed, next_norm.weight) if normed is not None else None), residual
+        out = ops.empty((T, self.w_out.shape[1]), dtype)
+        if self.padded:
+            out.zero_()
+        self._beside(fork, lambda: self.ffn.write_inner(y, out, 0))
+        self.mixer.write_inner(y, ctx, cache, out, self.mixer_column, 1.0)
+        self._join(fork)
+        return self._add(out, self.w_out, residual, next_norm), residual
+
+    def _add(self, out, weight, residual, next_norm):
+        ops = self.rt.ops
+        if self._plain_rms(next_norm) and getattr(next_norm, "deferrable", False) and getattr(ops, "fuses_next_norm", False):
+            return ops.linear_add(out, weight, residual, next_norm=(next_norm.weight, next_norm.eps))
+        return ops.linear_add(out, weight, residual)
+
+    @staticmethod
+    def _plain_rms(norm) -> bool:
+        return norm is not None and hasattr(norm, "deferrable")
+
+    def _beside(self, fork: bool, run):
+        if not fork:
+            return run()
+        stream = side_stream(self.rt)
+        ready = torch.cuda.Event()
+        ready.record(torch.cuda.current_stream(self.rt.device))
+        stream.wait_event(ready)
+        with torch.cuda.stream(stream):
+            return run()
+
+    def _join(self, fork: bool) -> None:
+        if fork:
+            torch.cuda.current_stream(self.rt.device).wait_stream(side_stream(self.rt))

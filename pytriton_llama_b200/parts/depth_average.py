@@ -22,17 +22,7 @@ from typing import Dict
 
 import torch
 
-from .base import Part, PartSpec, Runtime, TensorSpec, build_part, register_part
-
-
-class _Normed:
-    """The next block's first norm, already applied (what ``RMSNorm.forward`` passes through untouched)."""
-
-    def __init__(self, y: torch.Tensor, weight: torch.Tensor):
-        self.y, self.weight = y, weight
-
-    def materialise(self) -> torch.Tensor:
-        return self.y
+from .base import NormedInput, Part, PartSpec, Runtime, TensorSpec, build_part, register_part
 
 
 @register_part("block", "sandwich_depth_average")
@@ -102,4 +92,4 @@ class SandwichDepthAverageBlock(Part):
                                             next_weight=self.norm2.weight)
             y, residual = ops.post_norm_add([self.ffn.forward(y)], None, self.norm2b.weight, eps, residual, dtype=self.rt.dtype,
                                             **depth)
-        return (_Normed(y, following) if following is not None else None), residual
+        return (NormedInput(y, following) if following is not None else None), residual

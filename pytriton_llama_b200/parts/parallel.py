@@ -78,7 +78,7 @@ class ParallelMixers(Part):
         paged = [n for n in needs.values() if n.kind != "none"]
         if len(paged) > 1:
             raise ValueError("only one member of a parallel mixer may keep pages of keys and values")
-        states = tuple((f"{name}.{s}", shape) for name, n in needs.items() for s, shape in n.states)
+        states = tuple((f"{name}.{s}", *rest) for name, n in needs.items() for s, *rest in n.states)
         if any(n.state_shape is not None for n in needs.values()):
             raise ValueError("members of a parallel mixer name their states")
         base = paged[0] if paged else CacheNeed()

@@ -1,8 +1,9 @@
-"""Dense SwiGLU feed-forward.
+"""Dense gated feed-forward, SwiGLU or with another activation of the gate.
 
 lite_llama/models/llama.py:107-120: down(silu(gate(x)) * up(x)), three bias-free projections;
 silu(a) = a * sigmoid(a) in float32 (lite_llama/kernels/swiglu.py:44-46,64-66).  Gate and up are
-kept as one [2*inter, hidden] weight (gate rows first) so that one product feeds the activation.
+kept as one [2*inter, hidden] weight (gate rows first) so that one product feeds the activation.  ``act``
+"gelu_tanh" puts the tanh form of gelu in silu's place.
 """
 from __future__ import annotations
 
@@ -13,14 +14,18 @@ import torch
 from .base import Part, PartSpec, Runtime, TensorSpec, register_part
 
 
+@register_part("ffn", "gated_mlp")
 @register_part("ffn", "swiglu")
 class SwiGLU(Part):
-    """params: ``hidden``, ``inter``.  Tensors: ``gate``, ``up`` [inter, hidden], ``down`` [hidden, inter]."""
+    """params: ``hidden``, ``inter``, optional ``act`` ("silu" | "gelu_tanh").  Tensors: ``gate``, ``up`` [inter, hidden], ``down`` [hidden, inter]."""
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
         super().__init__(spec, runtime)
         self.hidden = int(spec.params["hidden"])
         self.inter = int(spec.params["inter"])
+        self.act = spec.params.get("act") or "silu"
+        if self.act not in ("silu", "gelu_tanh"):
+            raise ValueError(f"act={self.act!r} (known: silu, gelu_tanh)")
         self.w_gate_up = None
         self.w_down = None
 
@@ -48,12 +53,24 @@ class SwiGLU(Part):
         self.w_gate_up = self._to_compute(gu)
         self.w_down = self._to_compute(tensors["down"])
 
+    @property
+    def inner_width(self) -> int:
+        return self.inter
+
+    def write_inner(self, x, out, column: int) -> None:
+        """The input of the down projection into columns ``column``.. of ``out`` [T, >= column + inter]."""
+        ops = self.rt.ops
+        if self.alternating:
+            ops.gate_up_act(x, self.w_gate_up, self.act, out=out, column=column)
+        else:
+            ops.gated_act(ops.linear(x, self.w_gate_up), self.act, out=out, column=column)
+
     def forward(self, x, residual=None, next_norm=None):
         ops = self.rt.ops
         if self.alternating:
-            h = ops.gate_up_silu(x, self.w_gate_up)
+            h = ops.gate_up_act(x, self.w_gate_up, self.act)
         else:
-            h = ops.silu_mul(ops.linear(x, self.w_gate_up))
+            h = ops.gated_act(ops.linear(x, self.w_gate_up), self.act)
         if residual is not None:
             if next_norm is not None and getattr(ops, "fuses_next_norm", False):
                 return ops.linear_add(h, self.w_down, residual, next_norm=next_norm)

@@ -8,8 +8,9 @@ of their own size.  The nested ``position`` part then turns neighbouring pairs o
 or j < ``keep_first`` (``window`` 0: every j <= i); a kept key was rotated by its own position like any other.
 score = (q . k) * scale, softmax, heads of ``value_dim`` concatenated, W_o.
 
-Two options change the scores.  ``sink``: the softmax has one more term of score 0 in its denominator
-(a key that every query sees and that has no value), p_j = exp(s_j) / (1 + sum exp(s_j)).
+Two options change the scores.  ``sink``: the softmax has one more term in its denominator (a key that every query sees
+and that has no value), p_j = exp(s_j) / (exp(z) + sum exp(s_j)): with True z = 0, with "learned" z is a number per head
+(tensor ``sink``), which the scale does not touch.
 ``q_temp`` = {coef, every}: the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1);
 the factor is applied to the float32 scores, which is the same thing.
 
@@ -22,6 +23,9 @@ query i sees one key and one value for every block b of P positions with bP + P 
 block's keys (as the cache holds them) and values, in the same softmax; positions that the window has passed and
 whose block is not complete behind it are not seen.  The means are kept in pages of their own
 (``CacheNeed.pool_block``), written in the step that brings a block's last position.
+
+``bias``: the query and key projections (and the value projection) have biases.  ``values_are_keys``: there is no value
+projection, the value of a position is its key as projected, before it is turned; the cache keeps both.
 
 With ``own_kv`` False the layer has no key and value tensors: it attends, with its own queries and
 its own window, over the cache entry that another layer writes (``RunEntry.write`` False).
@@ -68,6 +72,20 @@ class RotaryPairs(Part):
             raise ValueError(f"rotary width {self.dims} must be even and at most the head size {self.head_dim}")
         f, self.amplitude = yarn_pair_frequencies(self.dims, float(p["base"]), p.get("scaling"))
         self.freq = f.to(torch.float32).to(runtime.device)
+        # the same table in 64 bits, one tensor for all layers with the same parameters: an operator set that works a
+        # step's angles out once tells tables apart by their address
+        scaling = p.get("scaling")
+        key = ("rotary_pairs", self.dims, float(p["base"]), tuple(sorted(scaling.items())) if scaling else None)
+        shared = getattr(runtime, "_shared_tables", None)
+        if shared is None:
+            shared = {}
+            try:
+                setattr(runtime, "_shared_tables", shared)
+            except AttributeError:          # (a runtime that takes no new attributes: every part keeps its own table)
+                pass
+        if key not in shared:
+            shared[key] = f.to(torch.float64).to(runtime.device)
+        self.freq64 = shared[key]
 
     def rotary_table(self):
         return None                      # not the split-halves rotation the fused cache-write kernels apply
@@ -75,14 +93,18 @@ class RotaryPairs(Part):
     def pair_table(self):
         return self.freq, self.dims, self.amplitude
 
+    def pair_table64(self):
+        """(float64 frequencies [dims/2], dims, amplitude)."""
+        return self.freq64, self.dims, self.amplitude
+
 
 @register_part("mixer", "window_attention")
 class WindowAttention(Part):
     """params: ``hidden``, ``heads``, ``kv_heads``, ``head_dim``, ``value_dim``, ``scale``, ``window``, ``keep_first``,
     ``qk_norm_eps``, ``own_kv``, ``sink``, ``q_temp``, ``qk_norm`` ("whole" | "per_head"), ``distance_bias``, ``gate`` (None | "sigmoid"),
-    ``pool``.  Nested part ``position`` (none: no encoding).  Tensors: ``q`` [heads*d, hidden], ``o`` [hidden,
+    ``pool``, ``bias``, ``values_are_keys``.  Nested part ``position`` (none: no encoding).  Tensors: ``q`` [heads*d, hidden], ``o`` [hidden,
     heads*value_dim], ``q.norm`` [heads*d]; with ``own_kv`` ``k`` [kv_heads*d, hidden], ``v`` [kv_heads*value_dim,
-    hidden], ``k.norm`` [kv_heads*d]."""
+    hidden] (not with ``values_are_keys``), ``k.norm`` [kv_heads*d]; ``q.b``, ``k.b``, ``v.b``; ``sink`` [heads]."""
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
         super().__init__(spec, runtime)
@@ -93,7 +115,16 @@ class WindowAttention(Part):
         self.window, self.keep_first = int(p.get("window") or 0), int(p.get("keep_first") or 0)
         self.qk_norm_eps = float(p.get("qk_norm_eps") or 0.0)
         self.own_kv = bool(p.get("own_kv", True))
-        self.sink = bool(p.get("sink", False))
+        self.sink = p.get("sink") or False
+        if self.sink not in (False, True, "learned"):
+            raise ValueError(f"sink={self.sink!r} (known: true, learned)")
+        self.bias, self.values_are_keys = bool(p.get("bias")), bool(p.get("values_are_keys"))
+        # biases and values out of the keys go through the kernel that turns pairs and writes the cache without a norm
+        self.plain_pairs = self.bias or self.values_are_keys
+        if self.plain_pairs and (self.qk_norm_eps > 0 or not self.own_kv or p.get("gate") or p.get("pool")):
+            raise ValueError("biases and values out of the keys go with neither a query/key norm, a gate, pooled blocks nor another layer's keys")
+        if self.values_are_keys and self.dv != self.d:
+            raise ValueError(f"values that are keys have the keys' size, not {self.dv} for {self.d}")
         temp = p.get("q_temp") or {}
         self.temp_coef, self.temp_every = float(temp.get("coef", 0.0)), int(temp.get("every", 1))
         self.per_head_norm = (p.get("qk_norm") or "whole") == "per_head"
@@ -109,7 +140,10 @@ class WindowAttention(Part):
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads are no multiple of {self.kv_heads} kv heads")
         self.position = build_part("position", spec.parts["position"], runtime) if "position" in spec.parts else None
-        self.w_in = self.w_o = self.q_norm = self.k_norm = None
+        if self.plain_pairs and self.position is not None and not hasattr(self.position, "pair_table64"):
+            raise ValueError("biases and values out of the keys go with a rotation of neighbouring pairs or with none")
+        self.inner_width = self.heads * self.dv
+        self.w_in = self.w_o = self.q_norm = self.k_norm = self.b_in = self.sink_scores = None
 
     def children(self):
         return {"position": self.position} if self.position is not None else {}
@@ -118,7 +152,14 @@ class WindowAttention(Part):
         H, G, d, dv = self.heads, self.kv_heads, self.d, self.dv
         out = {"q": TensorSpec((H * d, self.hidden)), "o": TensorSpec((self.hidden, H * dv))}
         if self.own_kv:
-            out.update({"k": TensorSpec((G * d, self.hidden)), "v": TensorSpec((G * dv, self.hidden))})
+            out["k"] = TensorSpec((G * d, self.hidden))
+            if not self.values_are_keys:
+                out["v"] = TensorSpec((G * dv, self.hidden))
+        if self.bias:
+            for name in [n for n in ("q", "k", "v") if n in out]:
+                out[name + ".b"] = TensorSpec((out[name].shape[0],), "zeros_jitter")
+        if self.sink == "learned":
+            out["sink"] = TensorSpec((H,), "zeros_jitter")
         if self.qk_norm_eps > 0:
             out["q.norm"] = TensorSpec((d if self.per_head_norm else H * d,), "ones_jitter")
             if self.own_kv:
@@ -128,7 +169,12 @@ class WindowAttention(Part):
         return out
 
     def load(self, t) -> None:
-        rows = [t["q"], t["k"], t["v"]] if self.own_kv else [t["q"]]
+        names = (["q", "k"] + ([] if self.values_are_keys else ["v"])) if self.own_kv else ["q"]
+        rows = [t[n] for n in names]
+        if self.bias:
+            self.b_in = self._to_f32(torch.cat([t[n + ".b"] for n in names], dim=0))
+        if self.sink == "learned":
+            self.sink_scores = self._to_f32(t["sink"])
         self.gate_column = sum(int(r.shape[0]) for r in rows)
         self.w_in = self._to_compute(torch.cat(rows + ([t["g"]] if self.gate else []), dim=0))
         self.w_o = self._to_compute(t["o"])
@@ -143,6 +189,15 @@ class WindowAttention(Part):
                          keep_first=self.keep_first if self.window else 0, pool_block=self.pool)
 
     def forward(self, x, ctx, cache):
+        return self.rt.ops.linear(self.heads_output(x, ctx, cache), self.w_o)
+
+    def write_inner(self, x, ctx, cache, out, column: int, scale: float = 1.0) -> None:
+        """The heads' outputs into columns ``column``.. of ``out`` [T, >= column + heads*value_dim]."""
+        if scale != 1.0:
+            raise ValueError("the heads' outputs are written as they are")
+        self.heads_output(x, ctx, cache, out=out, column=column)
+
+    def heads_output(self, x, ctx, cache, **where):
         ops = self.rt.ops
         g = cache.group
         if self.own_kv != bool(cache.write):
@@ -152,7 +207,11 @@ class WindowAttention(Part):
         if table is not None and table[1] and hasattr(self.position, "rotary_table64") and (self.per_head_norm or self.qk_norm_eps <= 0):
             table = self.position.rotary_table64()
         G = self.kv_heads if self.own_kv else 0
-        if table is not None and (self.per_head_norm or self.qk_norm_eps <= 0):
+        if self.plain_pairs:
+            freq, dims, amplitude = self.position.pair_table64() if self.position is not None else (None, 0, 1.0)
+            ops.pair_rotate_store(proj, self.heads, G, self.d, self.dv, self.b_in, ctx.positions, freq, dims, amplitude, g.slots,
+                                  cache.kv, g.page_size, values_are_keys=self.values_are_keys)
+        elif table is not None and (self.per_head_norm or self.qk_norm_eps <= 0):
             # halves of a head turned against each other (or nothing turned), a norm per head (or none)
             inv_freq, rot = table
             ops.head_norm_rotate_store(proj, self.heads, G, self.d, self.dv, self.q_norm, self.k_norm, self.qk_norm_eps,
@@ -165,7 +224,7 @@ class WindowAttention(Part):
             ops.qk_norm_rotate_store(proj, self.heads, G, self.d, self.dv, self.q_norm, self.k_norm,
                                      self.qk_norm_eps, ctx.positions, freq, dims, amplitude,
                                      g.slots if self.own_kv else None, cache.kv if self.own_kv else None, g.page_size)
-        extra = {}
+        extra = dict(where)
         if self.pool:
             sg = cache.summary_group
             if sg is None or cache.summary is None:
@@ -177,8 +236,7 @@ class WindowAttention(Part):
             extra["distance_bias"] = self.distance_bias
         if self.gate:
             extra["gate_column"] = self.gate_column
-        o = ops.window_attention(proj, cache.kv, g.block_table, ctx.tok_req, ctx.positions, self.heads, self.kv_heads, self.d,
-                                 self.dv, g.page_size, self.scale, window=self.window, keep_first=self.keep_first,
-                                 splits=ctx.attn_splits, hints=ctx, sink=self.sink, temp_coef=self.temp_coef,
-                                 temp_every=self.temp_every, **extra)
-        return ops.linear(o, self.w_o)
+        return ops.window_attention(proj, cache.kv, g.block_table, ctx.tok_req, ctx.positions, self.heads, self.kv_heads, self.d,
+                                    self.dv, g.page_size, self.scale, window=self.window, keep_first=self.keep_first,
+                                    splits=ctx.attn_splits, hints=ctx, sink=self.sink if self.sink_scores is None else self.sink_scores,
+                                    temp_coef=self.temp_coef, temp_every=self.temp_every, **extra)

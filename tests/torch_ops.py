@@ -55,9 +55,20 @@ class TorchOps:
         return False
 
     def silu_mul(self, gu):
+        return self.gated_act(gu, "silu")
+
+    def gated_act(self, gu, act, out=None, column=0):
         inter = gu.shape[1] // 2
-        g, u = gu[:, :inter].float(), gu[:, inter:].float()
-        return (g * torch.sigmoid(g) * u).to(gu.dtype)
+        g, u = gu[:, :inter].double(), gu[:, inter:].double()
+        if act == "silu":
+            g = g * torch.sigmoid(g)
+        else:
+            assert act == "gelu_tanh", act
+            g = 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3)))
+        if out is None:
+            return (g * u).to(gu.dtype)
+        out[:, column:column + inter] = (g * u).to(out.dtype)
+        return out
 
     def rope_kv_write(self, qkv, positions, inv_freq, rot, slots, cache, nq, nkv, d, page_size):
         T = qkv.shape[0]
@@ -145,6 +156,19 @@ class TorchOps:
             x[:, 0::2] += torch.sin(ang)
             x[:, 1::2] += torch.cos(ang)
         return x.float()
+
+    def embed_bigram(self, ids, table, scale, pairs, mul_prev, mul_cur, ctx, last):
+        buckets = pairs.shape[0] - 1
+        toks = ids.tolist()
+        rows = [buckets] * len(toks)
+        for lo, hi, slot, pos0 in self._requests(ctx):
+            before = int(last[slot, 0])
+            for t in range(lo, hi):
+                if pos0 + t - lo > 0:
+                    rows[t] = (before * mul_prev + toks[t] * mul_cur) % buckets
+                before = toks[t]
+            last[slot, 0] = before
+        return (table[ids.long()].double() * scale + pairs[torch.tensor(rows)].double()).float()
 
     def softcap(self, logits, cap):
         logits.copy_((cap * torch.tanh(logits.double() / cap)).float())
@@ -335,7 +359,12 @@ class TorchOps:
 
     def window_attention(self, q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window=0, keep_first=0,
                          splits=1, hints=None, sink=False, temp_coef=0.0, temp_every=1, shared_values=False, distance_bias=0.0,
-                         gate_column=-1, pool=0, summary=None, summary_table=None):
+                         gate_column=-1, pool=0, summary=None, summary_table=None, out=None, column=0):
+        if out is not None:
+            out[:, column:column + H * dv] = self.window_attention(
+                q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window, keep_first, splits, hints, sink, temp_coef,
+                temp_every, shared_values, distance_bias, gate_column, pool, summary, summary_table)
+            return out
         T = q.shape[0]
         out = torch.zeros((T, H * dv), dtype=torch.float64)
         group = H // G
@@ -370,16 +399,41 @@ class TorchOps:
                 sc = (k[:, h // group] @ qt[h]) * scale * temp
                 if distance_bias:
                     sc = sc - 2.0 ** (-distance_bias * (h + 1) / H) * dist
-                if sink:
-                    m = max(float(sc.max()), 0.0)
+                if isinstance(sink, torch.Tensor) or sink:
+                    z = float(sink[h]) if isinstance(sink, torch.Tensor) else 0.0      # the extra term's score
+                    m = max(float(sc.max()), z)
                     ex = torch.exp(sc - m)
-                    w = ex / (ex.sum() + math.exp(-m))
+                    w = ex / (ex.sum() + math.exp(z - m))
                 else:
                     w = torch.softmax(sc, 0)
                 out[t, h * dv:(h + 1) * dv] = w @ v[:, h // group]
         if gate_column >= 0:
             out = out * torch.sigmoid(q[:, gate_column:gate_column + H * dv].double())
         return out.to(q.dtype)
+
+    def pair_rotate_store(self, proj, H, G, d, dv, bias, positions, freq, dims, amplitude, slots, cache, page_size, values_are_keys=False):
+        """proj [T, q | k (| v)] + bias: neighbouring pairs of q (in place) and k turned, k and v (or k before it is turned)
+        to the cache."""
+        T = proj.shape[0]
+        x = proj.double()
+        if bias is not None:
+            x[:, :bias.numel()] += bias.double()
+        qk = x[:, :(H + G) * d].reshape(T, H + G, d).clone()
+        v = qk[:, H:].clone() if values_are_keys else x[:, (H + G) * d:(H + G) * d + G * dv].reshape(T, G, dv)
+        if freq is not None and dims > 0:
+            ang = positions.double()[:, None] * freq.double()[None, :dims // 2]
+            c, s = (ang.cos() * amplitude)[:, None, :], (ang.sin() * amplitude)[:, None, :]
+            a, b = qk[..., 0:dims:2].clone(), qk[..., 1:dims:2].clone()
+            qk[..., 0:dims:2] = a * c - b * s
+            qk[..., 1:dims:2] = b * c + a * s
+        proj[:, :H * d] = qk[:, :H].reshape(T, -1).to(proj.dtype)
+        for t in range(T):
+            sl = int(slots[t]) if cache is not None else -1
+            if sl >= 0:
+                page, off = divmod(sl, page_size)
+                kp, vp = self._page_views(cache, page, G, page_size, d, dv)
+                kp[:, off] = qk[t, H:].to(cache.dtype)
+                vp[:, off] = v[t].to(cache.dtype)
 
     def head_norm_rotate_store(self, proj, H, G, d, dv, q_norm, k_norm, eps, positions, inv_freq, rot, slots, cache, page_size):
         """proj [T, q | k | v | ...] in place: every q and k head divided by its own root mean square and multiplied by
@@ -476,15 +530,26 @@ class TorchOps:
         z = x.double()
         return (0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))).to(x.dtype)
 
-    def routed_experts(self, x, logits, w_gate_up, w_down, top, scale_input, shared, score="sigmoid", groups=1, keep_groups=1,
-                       renormalise=False):
+    def routed_experts(self, x, logits, w_gate_up, w_down, top, scale_input, shared, **routing):
+        out = torch.zeros((x.shape[0], w_down.shape[1]), dtype=torch.float64)
+        for t, y in self.expert_rows(x, logits, w_gate_up, w_down, top, scale_input, **routing):
+            out[t] += y
+        if shared is not None:
+            out += shared.double()
+        return out.float()
+
+    def expert_rows(self, x, logits, w_gate_up, w_down, top, scale_input=False, score="sigmoid", groups=1, keep_groups=1,
+                    renormalise=False, correction=None, weight_scale=1.0, clamped=None):
+        """[(token, weighted output of one of its choices)] in the order of the choices."""
         T = x.shape[0]
-        E = logits.shape[1]
+        E, real = logits.shape[1], w_gate_up.shape[0]
         inter = w_gate_up.shape[1] // 2
         score = torch.softmax(logits.double(), dim=-1) if score == "softmax" else torch.sigmoid(logits.double())
-        out = torch.zeros((T, w_down.shape[1]), dtype=torch.float64)
+        rows = []
         for t in range(T):
             allowed = score[t].clone()
+            if correction is not None:
+                allowed += correction.double()
             if groups > 1 and keep_groups < groups:
                 best = score[t].view(groups, E // groups).max(dim=1).values
                 kept = set(best.topk(keep_groups).indices.tolist())
@@ -494,15 +559,36 @@ class TorchOps:
             chosen = allowed.topk(top).indices.tolist()
             total = sum(score[t, e] for e in chosen) + 1e-20 if renormalise else 1.0
             for e in chosen:
-                w = score[t, e] / total
+                w = score[t, e] / total * weight_scale
+                if e >= real:               # an expert without weights hands its input on
+                    rows.append((t, w * x[t].double()))
+                    continue
                 u = (x[t].double() * w).to(x.dtype).double() if scale_input else x[t].double()
                 gu = w_gate_up[e].double() @ u
                 g, up = gu[:inter], gu[inter:]
-                y = w_down[e].double() @ (g * torch.sigmoid(g) * up)
-                out[t] += y if scale_input else w * y
-        if shared is not None:
-            out += shared.double()
-        return out.float()
+                if clamped is not None:
+                    limit, alpha, shift = clamped
+                    g, up = g.clamp(max=limit), up.clamp(-limit, limit)
+                    h = g * torch.sigmoid(alpha * g) * (up + shift)
+                else:
+                    h = g * torch.sigmoid(g) * up
+                y = w_down[e].double() @ h
+                rows.append((t, y if scale_input else w * y))
+        self._rows_of = x                   # (the type of what combine_experts_add returns)
+        return rows
+
+    def combine_experts_add(self, rows, residual, add=None, shared=None, next_norm=None):
+        s = residual.double()
+        for extra in (add, shared):
+            if extra is not None:
+                s = s + extra.double()
+        for t, y in rows:
+            s[t] += y
+        residual.copy_(s.float())
+        if next_norm is None:
+            return None
+        weight, eps = next_norm
+        return (s / torch.sqrt((s * s).mean(-1, keepdim=True) + eps) * weight.double()).to(self._rows_of.dtype)
 
     # ------------------------------------------------------------------ operators of the Sogalix parts
     def add_layernorm(self, x, residual, weight, bias, eps, rows=None, dtype=None, add_bias=None, keep_sum=True):
