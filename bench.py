@@ -5,6 +5,7 @@
     python bench.py --family lilenex      # likewise the Lilenex decoder
     python bench.py --family sogalix      # the Sogalix decoder beside a Lilenex and a Llama of equal size
     python bench.py --family podizen      # the Podizen decoder beside a Lilenex and a Llama of equal size
+    python bench.py --family nesisun      # the Nesisun decoder likewise
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and context 4096, timed on
 the device with CUDA events around exactly K decode steps (a step = the engine's step function for
@@ -239,13 +240,27 @@ def _podizen(width, layers, ff, vocab):
                        {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe} for i in range(layers)]}
 
 
+def _nesisun(width, layers, ff, vocab):
+    """A Nesisun of sizes that resemble a real model's layers, every layer with tensors of its own.  Attention with heads of
+    128, 4 query heads per kv head, half of every head rotated, a window of 1,024 positions that keeps the first 4; layers
+    alternate between a dense gated feed-forward of ff and 16 experts of ff/4 beside 2 that hand their input on, four
+    experts per token (about as many weights at work as the dense layer has)."""
+    heads = width // 128
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "mask": {"size": 1024, "keep_first": 4}, "rot": {"dims": 64, "base": 1000000.0}}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": 16, "identity": 2, "top": 4, "scale": 2.5}}
+    return {"architecture": "Nesisun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31337, "mul_cur": 7919}},
+            "layers": [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": ff} if i % 2 == 0 else moe} for i in range(layers)]}
+
+
 FAMILIES = {"tibepel": (_tibepel, ["llama"]), "lilenex": (_lilenex, ["llama"]), "sogalix": (_sogalix, ["lilenex", "llama"]),
-            "podizen": (_podizen, ["lilenex", "llama"])}
+            "podizen": (_podizen, ["lilenex", "llama"]), "nesisun": (_nesisun, ["lilenex", "llama"])}
 
 
 def family_bench(args) -> int:
-    """``--family tibepel``, ``lilenex``, ``sogalix`` or ``podizen``: prefill (one step of 2,048 prompt tokens, as one prompt and as 8 prompts of 256) and decode
-    (8 requests at 1,024 tokens, a step with its sampling kernel) of that decoder and of a Llama decoder (for Sogalix and Podizen also a Lilenex decoder) of the
+    """``--family tibepel``, ``lilenex``, ``sogalix``, ``podizen`` or ``nesisun``: prefill (one step of 2,048 prompt tokens, as one prompt and as 8 prompts of 256) and decode
+    (8 requests at 1,024 tokens, a step with its sampling kernel) of that decoder and of a Llama decoder (for Sogalix, Podizen and Nesisun also a Lilenex decoder) of the
     same width, depth, feed-forward size and vocabulary, on random weights, timed with CUDA events after warm-up; then one timed step of each kind with
     every operator bracketed by events, for the milliseconds by class of kernels.  One JSON line."""
     import torch
@@ -381,7 +396,7 @@ def main() -> int:
     ap.add_argument("--batch", type=int, default=None, help="decode batch (default: 8; 32 for 3b; 64 for 8b)")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the model has (named in config)")
     ap.add_argument("--points", default=None, help="extra decode batch sizes, comma separated ('' for none)")
-    ap.add_argument("--family", default=None, choices=["tibepel", "lilenex", "sogalix", "podizen"],
+    ap.add_argument("--family", default=None, choices=sorted(FAMILIES),
                     help="another workload: this decoder beside a Llama of equal size, prefill and decode (own JSON line)")
     ap.add_argument("--family-sizes", default=None, help="with --family: WIDTHxLAYERSxFF[,...] (default 1024x8x4096,2048x8x8192)")
     ap.add_argument("--no-e2e", action="store_true")
