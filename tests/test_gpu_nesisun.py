@@ -51,7 +51,7 @@ def _rand(gen, *shape, scale=1.0):
 
 # ---------------------------------------------------------------------------- the pair embedding
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("width,buckets,mul_prev,mul_cur", [(64, 61, 13, 5), (36, 1, 3, 2), (33, 509, 3_000_000_019, 1_000_003), (1032, 97, -7, 11)])
+@pytest.mark.parametrize("width,buckets,mul_prev,mul_cur", [(64, 61, 13, 5), (36, 1, 3, 2), (33, 401, 3_000_000_019, 1_000_003), (1032, 97, -7, 11)])
 def test_pair_embedding_and_the_last_tokens_state(ops, dtype, width, buckets, mul_prev, mul_cur):
     g = torch.Generator().manual_seed(width)
     dt, ref, vocab = DTYPES[dtype], TorchOps(), 70
@@ -90,7 +90,7 @@ def _paged(gen, q_lens, starts, page, pages, width):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,d,dv,page,dims,bias,from_keys", [
-    (4, 2, 64, 64, 16, 64, True, True), (6, 3, 48, 48, 8, 20, True, True), (3, 1, 7, 7, 4, 4, True, True), (8, 2, 128, 128, 16, 64, False, True),
+    (6, 2, 64, 64, 16, 64, True, True), (6, 3, 48, 48, 8, 20, True, True), (3, 1, 7, 7, 4, 4, True, True), (8, 2, 128, 128, 16, 64, False, True),
     (2, 2, 24, 24, 4, 0, True, True), (5, 1, 72, 40, 32, 72, True, False), (1, 1, 9, 5, 8, 2, False, False), (2, 1, 40, 40, 16, 38, True, True)])
 def test_bias_rotation_of_neighbours_and_values_from_keys(ops, dtype, H, G, d, dv, page, dims, bias, from_keys):
     g = torch.Generator().manual_seed(H * 100 + d)
@@ -117,7 +117,7 @@ def test_bias_rotation_of_neighbours_and_values_from_keys(ops, dtype, H, G, d, d
 
 # ---------------------------------------------------------------------------- attention with a learned sink
 SINK_SHAPES = [   # H, G, d, page, window, keep
-    (4, 2, 64, 16, 40, 20), (6, 3, 48, 8, 9, 30), (8, 2, 128, 16, 70, 3), (3, 3, 16, 4, 1, 2), (2, 1, 64, 16, 0, 0), (5, 1, 72, 32, 33, 7),
+    (6, 2, 64, 16, 45, 26), (6, 3, 48, 8, 9, 30), (8, 2, 128, 16, 70, 3), (3, 3, 16, 4, 1, 2), (2, 1, 64, 16, 0, 0), (5, 1, 72, 32, 33, 7),
     (4, 1, 128, 4, 64, 65), (2, 2, 7, 8, 5, 0),
 ]
 
@@ -235,7 +235,7 @@ def test_product_with_gated_activation_in_its_epilogue(ops, T, hidden, inter, ac
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("T,W,ff,E,identity,top,normed", [
-    (45, 64, 32, 8, 2, 3, True), (3, 96, 64, 16, 0, 1, True), (200, 48, 24, 6, 3, 4, False), (17, 40, 16, 1, 5, 2, True),
+    (45, 64, 32, 7, 3, 4, True), (3, 96, 64, 16, 0, 1, True), (200, 48, 24, 6, 3, 4, False), (17, 40, 16, 1, 5, 2, True),
     (300, 128, 96, 32, 8, 6, True), (5, 33, 8, 3, 1, 4, True), (9, 64, 16, 130, 20, 5, False), (2, 8, 8, 40, 10, 50, True), (1, 2048, 64, 4, 1, 2, True)])
 def test_clamped_experts_identity_correction_and_the_sum_with_the_next_norm(ops, dtype, T, W, ff, E, identity, top, normed):
     g = torch.Generator().manual_seed(T + E)
@@ -437,7 +437,7 @@ def _random_config(seed):
     for _ in range(rng.randint(0, 3)):
         layers.append(plain.again(layers, rng.randrange(own)))
     return plain.config(rng.randint(50, 300), width, layers, eps=rng.choice([1e-6, 1e-5, 1e-3]), scale=rng.choice([0.5, 1.0, 1.4]),
-                        buckets=rng.choice([1, 7, 509, 4001]), mul_prev=rng.randint(1, 10000), mul_cur=rng.randint(1, 10000))
+                        buckets=rng.choice([1, 7, 401, 4001]), mul_prev=rng.randint(1, 10000), mul_cur=rng.randint(1, 10000))
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
