@@ -1,6 +1,7 @@
 from .llama import ConfigError, LlamaConfig, RopeScaling  # noqa: F401
 from .engine import EngineConfig  # noqa: F401
 from .tibepel import TibepelConfig  # noqa: F401
+from .gepilix import GepilixConfig  # noqa: F401
 from .lilenex import LilenexConfig  # noqa: F401
 from .sogalix import SogalixConfig  # noqa: F401
 from .nesisun import NesisunConfig  # noqa: F401

@@ -67,6 +67,9 @@ def _register_builtin() -> None:
     from .nesisun import NesisunConfig
     from ..models.nesisun import nesisun_spec
     register_architecture("Nesisun", NesisunConfig.from_dict, nesisun_spec)
+    from .gepilix import GepilixConfig
+    from ..models.gepilix import gepilix_spec
+    register_architecture("Gepilix", GepilixConfig.from_dict, gepilix_spec)
 
 
 _register_builtin()

@@ -29,6 +29,9 @@ Contracts (``T`` = tokens of the step, all tensors on the runtime's device):
   ``output_bias`` (float32 [H] or None): whoever adds the output into the stream adds it too;
 * token_input: ``apply(residual, x, bias, ctx)`` adds ``x`` (+ ``bias``), then its own term, into
   the float32 ``residual`` in place;
+* a mixer or ffn with the class attribute ``takes_tail = True`` may be called with ``tail=<Tail>``: it hands the last
+  thing it computes to the tail, which adds it (times the layer's scale) into the stream and returns the next norm's
+  result, and returns what the tail returns;
 * a mixer or ffn with the class attribute ``fuses_residual = True`` is called with
   ``residual=<float32 [T, H]>`` as well and may add its output into it and return None;
 * embedding: ``cache_need() -> CacheNeed`` of kind "none" (its per-request states);
@@ -159,6 +162,38 @@ class NormedInput:
 
     def materialise(self) -> torch.Tensor:
         return self.y
+
+
+class ScaledOutput:
+    """A sub-layer's output that the next norm has to multiply by ``scale`` (float32 [H]) when it adds it."""
+
+    def __init__(self, x: torch.Tensor, scale: torch.Tensor):
+        self.x, self.scale = x, scale
+
+
+class Tail:
+    """What stands between a sub-layer's last step and the next sub-layer's input: residual <- residual + scale * output
+    and the norm that follows.  Each method takes another form of the last step and returns the normed input (``norm``:
+    the norm part, whose ``tail_add``, ``tail_product``, ``tail_members`` and ``tail_experts`` do the work)."""
+
+    def __init__(self, norm, residual: torch.Tensor, scale: torch.Tensor):
+        self.norm, self.residual, self.scale = norm, residual, scale
+
+    def output(self, out: torch.Tensor):
+        """The output itself."""
+        return self.norm.tail_add(out, self.residual, self.scale)
+
+    def product(self, inner: torch.Tensor, w: torch.Tensor):
+        """The output is inner @ w^T."""
+        return self.norm.tail_product(inner, w, self.residual, self.scale)
+
+    def members(self, outs, eps: float):
+        """The output is the mean of [(x, weight)], each x divided by its root mean square and multiplied by its weight."""
+        return self.norm.tail_members(outs, eps, self.residual, self.scale)
+
+    def experts(self, rows, shared):
+        """The output is the weighted sum of the chosen experts' outputs, plus ``shared`` (or None)."""
+        return self.norm.tail_experts(rows, shared, self.residual, self.scale)
 
 
 def side_stream(runtime: Runtime) -> "torch.cuda.Stream":

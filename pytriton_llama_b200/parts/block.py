@@ -3,8 +3,9 @@
 lite_llama/models/llama.py:136-162: pre-norm block.  The stream is carried as two tensors: the
 output of the last sub-layer (not yet added) and the float32 residual; each norm first adds the
 former into the latter.  The block returns its feed-forward output un-added, so the next block's
-first norm (or the model's final norm, :219) folds it in.  ``SharedNormBlock`` is the arrangement with one
-norm whose output both sub-layers read.
+first norm (or the model's final norm, :219) folds it in.  With a scale per sub-layer the block completes the
+stream itself and hands the next norm's result on.  ``SharedNormBlock`` is the arrangement with one norm whose
+output both sub-layers read.
 """
 from __future__ import annotations
 
@@ -12,13 +13,18 @@ import os
 
 import torch
 
-from .base import NormedInput, Part, PartSpec, Runtime, build_part, register_part, side_stream
+from .base import (NormedInput, Part, PartSpec, Runtime, ScaledOutput, Tail, TensorSpec, build_part, register_part,
+                   side_stream)
 
 
 @register_part("block", "pre_norm")
 class PreNormBlock(Part):
     """Nested parts: ``norm1``, ``mixer``; ``norm2`` and ``ffn`` (both or neither: a layer without a
-    feed-forward); optionally ``token_input``, which comes last."""
+    feed-forward); optionally ``token_input``, which comes last.
+
+    params: optional ``layer_scale`` (the stream's width): each sub-layer's result is multiplied entry by entry by a
+    vector before it is added, tensors ``scale1`` (mixer) and ``scale2`` (feed-forward).  The norms are then of a kind
+    with ``tail_add`` and the like (``tanh_norm``)."""
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
         super().__init__(spec, runtime)
@@ -32,6 +38,10 @@ class PreNormBlock(Part):
         last = self.ffn if self.ffn is not None else self.mixer
         if self.token_input is None and getattr(last, "output_bias_spec", False):
             raise ValueError("a block whose last projection leaves its bias out needs a token_input that adds it")
+        self.scale_width = int(spec.params.get("layer_scale") or 0)
+        self.scale1 = self.scale2 = None
+        if self.scale_width and (self.token_input is not None or not hasattr(self.norm1, "tail_add")):
+            raise ValueError("a layer scale goes with norms that add a scaled output, and with no token_input")
 
     takes_next_norm = True   # forward() accepts the norm part that follows the block
 
@@ -39,8 +49,39 @@ class PreNormBlock(Part):
         parts = {"norm1": self.norm1, "mixer": self.mixer, "norm2": self.norm2, "ffn": self.ffn, "token_input": self.token_input}
         return {k: v for k, v in parts.items() if v is not None}
 
+    def tensor_specs(self):
+        if not self.scale_width:
+            return {}
+        # drawn at random: around one, so that a scale that is left out or swapped shows
+        names = ["scale1"] + (["scale2"] if self.ffn is not None else [])
+        return {n: TensorSpec((self.scale_width,), "uniform", lo=0.5, hi=1.5) for n in names}
+
+    def load(self, tensors) -> None:
+        if self.scale_width:
+            self.scale1 = self._to_f32(tensors["scale1"])
+            self.scale2 = self._to_f32(tensors["scale2"]) if self.ffn is not None else None
+
     def cache_need(self):
         return self.mixer.cache_need()
+
+    def _forward_scaled(self, x, residual, ctx, cache, next_norm):
+        y, residual = self.norm1.forward(x, residual)
+        y = self._run_scaled(self.mixer, y, residual, self.scale1, self.norm2 if self.ffn is not None else next_norm, ctx, cache)
+        if self.ffn is not None:
+            y, _ = self.norm2.forward(y, residual)
+            y = self._run_scaled(self.ffn, y, residual, self.scale2, next_norm)
+        return y, residual
+
+    @staticmethod
+    def _run_scaled(part, y, residual, scale, following, *args):
+        """``part``'s output times ``scale`` into the stream, and the following norm's result; without a norm that
+        follows (the model's last layer) the output and its scale, for the final norm to add to the rows it takes."""
+        if not hasattr(following, "tail_add"):
+            return ScaledOutput(part.forward(y, *args), scale)
+        tail = Tail(following, residual, scale)
+        if getattr(part, "takes_tail", False):
+            return NormedInput(part.forward(y, *args, tail=tail), following.weight)
+        return NormedInput(tail.output(part.forward(y, *args)), following.weight)
 
     def forward(self, x, residual, ctx, cache, next_norm=None):
         """``x`` may be None: the previous sub-layer then already added its output into ``residual``.
@@ -48,6 +89,8 @@ class PreNormBlock(Part):
         Those that also set ``emits_normed`` are told which norm reads the residual next
         (``next_norm``: the norm part that follows this block, if any) and may return that norm's
         prepared input; a sub-layer reads such an input only if it sets ``accepts_normed``."""
+        if self.scale_width:
+            return self._forward_scaled(x, residual, ctx, cache, next_norm)
         y, residual = self.norm1.forward(x, residual)
         a = self._run(self.mixer, y, residual, self.norm2, ctx, cache)
         bias = getattr(self.mixer, "output_bias", None)

@@ -1,5 +1,6 @@
 """Dense feed-forwards with one hidden layer, W_down act(W_up h), the activation worked out in float32.
 
+``relu2_mlp``: the square of max(z, 0).
 ``gelu_mlp``: the tanh form of gelu, gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
 ``xielu_mlp``: xIELU with two learned numbers (p, q) per layer: for z > 0, softplus(p) z^2 + z / 2; for z <= 0,
 (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2."""
@@ -46,3 +47,15 @@ class XieluMLP(GeluMLP):
     def forward(self, x):
         ops = self.rt.ops
         return ops.linear(ops.xielu(ops.linear(x, self.w_up), self.pos_factor, self.neg_factor), self.w_down)
+
+
+@register_part("ffn", "relu2_mlp")
+class SquaredReluMLP(GeluMLP):
+    """params: ``hidden``, ``inter``.  Tensors: ``up`` [inter, hidden], ``down`` [hidden, inter]."""
+
+    takes_tail = True
+
+    def forward(self, x, tail=None):
+        ops = self.rt.ops
+        inner = ops.linear_relu2(x, self.w_up)
+        return ops.linear(inner, self.w_down) if tail is None else tail.product(inner, self.w_down)

@@ -108,8 +108,12 @@ class ParallelMixers(Part):
                 main.wait_stream(stream)
         return [(outs[name], self.out_weights[name]) for name in names]
 
-    def forward(self, x, ctx, cache):
+    takes_tail = True
+
+    def forward(self, x, ctx, cache, tail=None):
         ops = self.rt.ops
+        if self.normed and tail is not None:
+            return tail.members(self.member_outputs(x, ctx, cache), self.norm_eps)
         if self.normed:
             return ops.mean_of_normed(self.member_outputs(x, ctx, cache), self.norm_eps, self.rt.dtype)
         joint = ops.empty((x.shape[0], self.inner_width), self.rt.dtype)
@@ -119,7 +123,7 @@ class ParallelMixers(Part):
         if not side_by_side:
             for name in names:
                 self.members[name].write_inner(x, ctx, cache.member(name), joint, self.columns[name], self.scales[name])
-            return ops.linear(joint, self.w_o)
+            return self._project(joint, tail)
         if self._streams is None:
             self._streams = [torch.cuda.Stream(self.rt.device) for _ in names[1:]]
         main = torch.cuda.current_stream(self.rt.device)
@@ -132,4 +136,11 @@ class ParallelMixers(Part):
         self.members[names[0]].write_inner(x, ctx, cache.member(names[0]), joint, self.columns[names[0]], self.scales[names[0]])
         for stream in self._streams:
             main.wait_stream(stream)
-        return ops.linear(joint, self.w_o)
+        return self._project(joint, tail)
+
+    def _project(self, joint, tail):
+        if tail is None:
+            return self.rt.ops.linear(joint, self.w_o)
+        if self.output_bias is not None:
+            raise ValueError("an output bias is added by the caller, not by a tail")
+        return tail.product(joint, self.w_o)

@@ -37,6 +37,18 @@ def rope_inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict
     return torch.where(in_band, blended, divided)
 
 
+def rope_frequencies64(theta: float, scaling: Optional[dict], rot: int) -> torch.Tensor:
+    """The same table worked out in float64 throughout."""
+    f = float(theta) ** (-torch.arange(0, rot, 2, dtype=torch.float64) / rot)
+    if scaling is None or scaling.get("rope_type", "default") == "default":
+        return f
+    factor, low, high = float(scaling["factor"]), float(scaling["low_freq_factor"]), float(scaling["high_freq_factor"])
+    turns = float(scaling["original_max_position_embeddings"]) * f / (2 * math.pi)      # original / wavelength
+    blend = (turns - low) / (high - low) if high != low else torch.ones_like(f)
+    mixed = (1 - blend) * f / factor + blend * f
+    return torch.where(turns > high, f, torch.where(turns < low, f / factor, mixed))
+
+
 @register_part("position", "rope")
 class RotaryPosition(Part):
     """params: ``head_dim``, ``theta``, ``scaling`` (None or the llama3 block), optional ``rotary_dim``."""
@@ -62,15 +74,10 @@ class RotaryPosition(Part):
         if key not in shared:
             shared[key] = rope_inverse_frequencies(self.head_dim, float(p["theta"]), scaling, self.rot).to(runtime.device)
         self.inv_freq = shared[key]
-        # the same frequencies in 64 bits, for kernels that work the angle out in 64 bits (an unscaled table is made
-        # anew from theta; a scaled one is the float32 table widened)
+        # the same frequencies in 64 bits, for kernels that work the angle out in 64 bits
         key64 = key + ("f64",)
         if key64 not in shared:
-            if scaling is None or scaling.get("rope_type", "default") == "default":
-                exact = float(p["theta"]) ** (-torch.arange(0, self.rot, 2, dtype=torch.float64) / self.rot)
-            else:
-                exact = self.inv_freq.detach().cpu().to(torch.float64)
-            shared[key64] = exact.to(runtime.device)
+            shared[key64] = rope_frequencies64(float(p["theta"]), scaling, self.rot).to(runtime.device)
         self.inv_freq64 = shared[key64]
 
     def rotary_table64(self) -> Tuple[torch.Tensor, int]:

@@ -10,7 +10,8 @@ Options of the router.  ``score`` "softmax": score = softmax(z) over all experts
 that many groups of neighbours, a group's score is its largest score, and only experts of the ``keep_groups`` groups
 with the largest scores can be chosen.  ``renormalise``: the weights are the chosen scores divided by their sum
 (+ 1e-20).  ``correction``: a number per expert that is added to the scores when experts are chosen, but not to their
-weights (tensor ``correction``).  ``weight_scale`` multiplies the weights.  ``identity`` = n: the router has n more
+weights (tensor ``correction``).  ``router_bias``: a number per expert that is added to its logit (tensor ``router.b``).
+``weight_scale`` multiplies the weights.  ``identity`` = n: the router has n more
 outputs, whose experts have no weights and hand their input on.  ``clamped`` = (limit, alpha, shift): an expert is
 W_down (min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + shift)) of g = W_gate h, u = W_up h.
 
@@ -33,8 +34,8 @@ from .base import Part, PartSpec, Runtime, TensorSpec, register_part
 @register_part("ffn", "routed_experts")
 class RoutedExperts(Part):
     """params: ``hidden``, ``inter``, ``experts``, ``top``, ``shared_inter`` (0: none), ``scale_input``, ``score`` ("sigmoid" |
-    "softmax"), ``groups``, ``keep_groups``, ``renormalise``, ``correction``, ``weight_scale``, ``identity``, ``clamped``.
-    Tensors: ``router`` [experts + identity, hidden]; ``correction`` [experts + identity]; per expert i ``e<i>.gate``, ``e<i>.up`` [inter, hidden], ``e<i>.down``
+    "softmax"), ``groups``, ``keep_groups``, ``renormalise``, ``correction``, ``router_bias``, ``weight_scale``, ``identity``, ``clamped``.
+    Tensors: ``router`` [experts + identity, hidden]; ``correction``, ``router.b`` [experts + identity]; per expert i ``e<i>.gate``, ``e<i>.up`` [inter, hidden], ``e<i>.down``
     [hidden, inter]; ``shared.gate``, ``shared.up`` [shared_inter, hidden], ``shared.down`` [hidden, shared_inter]."""
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
@@ -60,6 +61,7 @@ class RoutedExperts(Part):
         if self.score != "sigmoid" or self.groups > 1 or self.renormalise:
             self.routing = dict(score=self.score, groups=self.groups, keep_groups=self.keep_groups, renormalise=self.renormalise)
         self.has_correction = bool(p.get("correction", False))
+        self.has_router_bias = bool(p.get("router_bias", False))
         self.weight_scale = float(p.get("weight_scale", 1.0))
         self.clamped = tuple(float(v) for v in p["clamped"]) if p.get("clamped") else None
         if self.weight_scale != 1.0:
@@ -77,6 +79,8 @@ class RoutedExperts(Part):
         out = {"router": TensorSpec((self.experts + self.identity, self.hidden))}
         if self.has_correction:
             out["correction"] = TensorSpec((self.experts + self.identity,), "uniform", lo=-0.02, hi=0.02)
+        if self.has_router_bias:
+            out["router.b"] = TensorSpec((self.experts + self.identity,), "zeros_jitter")
         for i in range(self.experts):
             out.update({f"e{i}.gate": TensorSpec((self.inter, self.hidden)), f"e{i}.up": TensorSpec((self.inter, self.hidden)),
                         f"e{i}.down": TensorSpec((self.hidden, self.inter))})
@@ -90,6 +94,8 @@ class RoutedExperts(Part):
         self.w_router = self._to_compute(t["router"])
         if self.has_correction:
             self.routing["correction"] = self._to_f32(t["correction"])
+        if self.has_router_bias:
+            self.routing["logit_bias"] = self._to_f32(t["router.b"])
         # per expert the gate rows, then the up rows: one grouped product feeds the activation
         self.w_gate_up = self._to_compute(torch.stack([torch.cat([t[f"e{i}.gate"], t[f"e{i}.up"]], dim=0) for i in E]))
         self.w_down = self._to_compute(torch.stack([t[f"e{i}.down"] for i in E]))
@@ -128,10 +134,15 @@ class RoutedExperts(Part):
         rows, shared = begun
         return self.rt.ops.combine_experts_add(rows, residual, add=add, shared=shared, next_norm=next_norm)
 
-    def forward(self, x):
+    takes_tail = True
+
+    def forward(self, x, tail=None):
         ops = self.rt.ops
         if self.identity:
             raise ValueError("identity experts are added up by finish()")
+        if tail is not None and not self.scale_input:
+            return tail.experts(*self.begin(x))
         shared = self._shared_output(x)
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
-        return ops.routed_experts(x, logits, self.w_gate_up, self.w_down, self.top, self.scale_input, shared, **self.routing)
+        out = ops.routed_experts(x, logits, self.w_gate_up, self.w_down, self.top, self.scale_input, shared, **self.routing)
+        return out if tail is None else tail.output(out)

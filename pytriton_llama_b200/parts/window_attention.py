@@ -27,6 +27,10 @@ whose block is not complete behind it are not seen.  The means are kept in pages
 ``bias``: the query and key projections (and the value projection) have biases.  ``values_are_keys``: there is no value
 projection, the value of a position is its key as projected, before it is turned; the cache keeps both.
 
+``softcap`` = c > 0: a score s becomes c * tanh(s / c) before the softmax.  ``chunk`` = n > 0 (in a window's place): query i
+sees key j <= i if both lie in the same block of n positions, blocks counted from position 0 of the request.  ``gate``
+"head": head h's output is multiplied by sigmoid((W_g h)_h), one number per head.
+
 With ``own_kv`` False the layer has no key and value tensors: it attends, with its own queries and
 its own window, over the cache entry that another layer writes (``RunEntry.write`` False).
 """
@@ -102,9 +106,10 @@ class RotaryPairs(Part):
 class WindowAttention(Part):
     """params: ``hidden``, ``heads``, ``kv_heads``, ``head_dim``, ``value_dim``, ``scale``, ``window``, ``keep_first``,
     ``qk_norm_eps``, ``own_kv``, ``sink``, ``q_temp``, ``qk_norm`` ("whole" | "per_head"), ``distance_bias``, ``gate`` (None | "sigmoid"),
-    ``pool``, ``bias``, ``values_are_keys``.  Nested part ``position`` (none: no encoding).  Tensors: ``q`` [heads*d, hidden], ``o`` [hidden,
+    ``pool``, ``bias``, ``values_are_keys``, ``softcap``, ``chunk``.  Nested part ``position`` (none: no encoding).  Tensors: ``q`` [heads*d, hidden], ``o`` [hidden,
     heads*value_dim], ``q.norm`` [heads*d]; with ``own_kv`` ``k`` [kv_heads*d, hidden], ``v`` [kv_heads*value_dim,
-    hidden] (not with ``values_are_keys``), ``k.norm`` [kv_heads*d]; ``q.b``, ``k.b``, ``v.b``; ``sink`` [heads]."""
+    hidden] (not with ``values_are_keys``), ``k.norm`` [kv_heads*d]; ``q.b``, ``k.b``, ``v.b``; ``sink`` [heads]; ``g`` [heads*value_dim, hidden], or [heads, hidden]
+    with one gate per head."""
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
         super().__init__(spec, runtime)
@@ -121,8 +126,8 @@ class WindowAttention(Part):
         self.bias, self.values_are_keys = bool(p.get("bias")), bool(p.get("values_are_keys"))
         # biases and values out of the keys go through the kernel that turns pairs and writes the cache without a norm
         self.plain_pairs = self.bias or self.values_are_keys
-        if self.plain_pairs and (self.qk_norm_eps > 0 or not self.own_kv or p.get("gate") or p.get("pool")):
-            raise ValueError("biases and values out of the keys go with neither a query/key norm, a gate, pooled blocks nor another layer's keys")
+        if self.plain_pairs and (self.qk_norm_eps > 0 or not self.own_kv or p.get("pool")):
+            raise ValueError("biases and values out of the keys go with neither a query/key norm, pooled blocks nor another layer's keys")
         if self.values_are_keys and self.dv != self.d:
             raise ValueError(f"values that are keys have the keys' size, not {self.dv} for {self.d}")
         temp = p.get("q_temp") or {}
@@ -132,8 +137,11 @@ class WindowAttention(Part):
             raise ValueError(f"qk_norm={p.get('qk_norm')!r} (known: whole, per_head)")
         self.distance_bias = float(p.get("distance_bias") or 0.0)
         self.gate = p.get("gate") or None
-        if self.gate not in (None, "sigmoid"):
-            raise ValueError(f"gate={self.gate!r} (known: sigmoid)")
+        if self.gate not in (None, "sigmoid", "head"):
+            raise ValueError(f"gate={self.gate!r} (known: sigmoid, head)")
+        self.softcap, self.chunk = float(p.get("softcap") or 0.0), int(p.get("chunk") or 0)
+        if self.chunk and (self.window or not self.own_kv):
+            raise ValueError("blocks of positions go with neither a window nor another layer's keys")
         self.pool = int(p.get("pool") or 0) if self.window else 0
         if self.pool and (self.keep_first or not self.own_kv or self.sink):
             raise ValueError("pooled blocks go with neither kept first positions, a sink, nor another layer's keys")
@@ -143,6 +151,7 @@ class WindowAttention(Part):
         if self.plain_pairs and self.position is not None and not hasattr(self.position, "pair_table64"):
             raise ValueError("biases and values out of the keys go with a rotation of neighbouring pairs or with none")
         self.inner_width = self.heads * self.dv
+        self.output_bias = None
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.b_in = self.sink_scores = None
 
     def children(self):
@@ -165,7 +174,7 @@ class WindowAttention(Part):
             if self.own_kv:
                 out["k.norm"] = TensorSpec((d if self.per_head_norm else G * d,), "ones_jitter")
         if self.gate:
-            out["g"] = TensorSpec((H * dv, self.hidden))
+            out["g"] = TensorSpec((H if self.gate == "head" else H * dv, self.hidden))
         return out
 
     def load(self, t) -> None:
@@ -176,7 +185,11 @@ class WindowAttention(Part):
         if self.sink == "learned":
             self.sink_scores = self._to_f32(t["sink"])
         self.gate_column = sum(int(r.shape[0]) for r in rows)
-        self.w_in = self._to_compute(torch.cat(rows + ([t["g"]] if self.gate else []), dim=0))
+        if self.gate:
+            rows.append(t["g"])
+        if self.gate == "head":         # a projection's rows keep starting on 16-byte boundaries
+            rows.append(torch.zeros((-sum(int(r.shape[0]) for r in rows) % 8, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = self._to_compute(torch.cat(rows, dim=0))
         self.w_o = self._to_compute(t["o"])
         if self.qk_norm_eps > 0:
             self.q_norm = self._to_f32(t["q.norm"])
@@ -184,18 +197,16 @@ class WindowAttention(Part):
 
     def cache_need(self) -> CacheNeed:
         # (a block's mean is made in the step that brings its last position, from keys that must still be held then)
-        return CacheNeed(kind="window" if self.window else "full", kv_heads=self.kv_heads, head_dim=self.d,
-                         window=max(self.window, self.pool), value_dim=self.dv if self.dv != self.d else 0,
+        return CacheNeed(kind="window" if self.window else "chunk" if self.chunk else "full", kv_heads=self.kv_heads, head_dim=self.d,
+                         window=max(self.window, self.pool, self.chunk), value_dim=self.dv if self.dv != self.d else 0,
                          keep_first=self.keep_first if self.window else 0, pool_block=self.pool)
 
     def forward(self, x, ctx, cache):
         return self.rt.ops.linear(self.heads_output(x, ctx, cache), self.w_o)
 
     def write_inner(self, x, ctx, cache, out, column: int, scale: float = 1.0) -> None:
-        """The heads' outputs into columns ``column``.. of ``out`` [T, >= column + heads*value_dim]."""
-        if scale != 1.0:
-            raise ValueError("the heads' outputs are written as they are")
-        self.heads_output(x, ctx, cache, out=out, column=column)
+        """The heads' outputs, times ``scale``, into columns ``column``.. of ``out`` [T, >= column + heads*value_dim]."""
+        self.heads_output(x, ctx, cache, out=out, column=column, **({"out_scale": scale} if scale != 1.0 else {}))
 
     def heads_output(self, x, ctx, cache, **where):
         ops = self.rt.ops
@@ -236,6 +247,12 @@ class WindowAttention(Part):
             extra["distance_bias"] = self.distance_bias
         if self.gate:
             extra["gate_column"] = self.gate_column
+        if self.gate == "head":
+            extra["gate_per_head"] = True
+        if self.softcap > 0:
+            extra["softcap"] = self.softcap
+        if self.chunk:
+            extra["chunk"] = self.chunk
         return ops.window_attention(proj, cache.kv, g.block_table, ctx.tok_req, ctx.positions, self.heads, self.kv_heads, self.d,
                                     self.dv, g.page_size, self.scale, window=self.window, keep_first=self.keep_first,
                                     splits=ctx.attn_splits, hints=ctx, sink=self.sink if self.sink_scores is None else self.sink_scores,

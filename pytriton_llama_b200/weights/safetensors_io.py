@@ -111,4 +111,4 @@ def write_file(path: Union[str, Path], tensors: Dict[str, torch.Tensor]) -> None
         for name in order:
             t = tensors[name].detach().cpu().contiguous()
             if t.numel():
-                f.write(memoryview(t.view(torch.uint8).reshape(-1).numpy()))      # no copy of the tensor's bytes
+                f.write(memoryview(t.reshape(-1).view(torch.uint8).numpy()))      # no copy of the tensor's bytes

@@ -180,7 +180,7 @@ class TorchOps:
             if qs[r + 1] > qs[r]:
                 yield qs[r], qs[r + 1], int(ctx.state_slot[r]), int(ctx.positions[qs[r]])
 
-    def causal_conv(self, x, column, channels, w, b, state, ctx, silu=True):
+    def causal_conv(self, x, column, channels, w, b, state, ctx, silu=True, in_bias=None):
         taps = w.shape[1]
         out = torch.zeros((x.shape[0], channels), dtype=torch.float64)
         for lo, hi, slot, pos0 in self._requests(ctx):
@@ -188,7 +188,10 @@ class TorchOps:
             for j in range(taps - 1):            # entry j is the input at position pos0 - (taps - 1) + j: nothing before position 0
                 if pos0 - (taps - 1) + j < 0:
                     past[j] = 0
-            seq = torch.cat([past, x[lo:hi, column:column + channels].double()], 0)
+            new = x[lo:hi, column:column + channels].double()
+            if in_bias is not None:
+                new = new + in_bias.double()
+            seq = torch.cat([past, new], 0)
             for k in range(taps):
                 out[lo:hi] += seq[k:k + hi - lo] * w[:, k].double()
             if taps > 1:
@@ -359,11 +362,13 @@ class TorchOps:
 
     def window_attention(self, q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window=0, keep_first=0,
                          splits=1, hints=None, sink=False, temp_coef=0.0, temp_every=1, shared_values=False, distance_bias=0.0,
-                         gate_column=-1, pool=0, summary=None, summary_table=None, out=None, column=0):
+                         gate_column=-1, pool=0, summary=None, summary_table=None, out=None, column=0, softcap=0.0, chunk=0,
+                         gate_per_head=False, out_scale=1.0):
         if out is not None:
             out[:, column:column + H * dv] = self.window_attention(
                 q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window, keep_first, splits, hints, sink, temp_coef,
-                temp_every, shared_values, distance_bias, gate_column, pool, summary, summary_table)
+                temp_every, shared_values, distance_bias, gate_column, pool, summary, summary_table, softcap=softcap, chunk=chunk,
+                gate_per_head=gate_per_head, out_scale=out_scale)
             return out
         T = q.shape[0]
         out = torch.zeros((T, H * dv), dtype=torch.float64)
@@ -373,6 +378,8 @@ class TorchOps:
             if r < 0:
                 continue
             keys = [j for j in range(p + 1) if not window or p - j < window or j < keep_first]
+            if chunk:
+                keys = [j for j in keys if j // chunk == p // chunk]
             ks, vs = [], []
             n_blocks = max(0, (p - window + 1) // pool) if pool and window else 0     # blocks that lie wholly behind the window
             for b in range(n_blocks):
@@ -397,6 +404,8 @@ class TorchOps:
             dist = torch.tensor([0.0] * n_blocks + [float(p - j) for j in keys], dtype=torch.float64)
             for h in range(H):
                 sc = (k[:, h // group] @ qt[h]) * scale * temp
+                if softcap:
+                    sc = softcap * torch.tanh(sc / softcap)
                 if distance_bias:
                     sc = sc - 2.0 ** (-distance_bias * (h + 1) / H) * dist
                 if isinstance(sink, torch.Tensor) or sink:
@@ -407,9 +416,11 @@ class TorchOps:
                 else:
                     w = torch.softmax(sc, 0)
                 out[t, h * dv:(h + 1) * dv] = w @ v[:, h // group]
-        if gate_column >= 0:
+        if gate_column >= 0 and gate_per_head:
+            out = out * torch.sigmoid(q[:, gate_column:gate_column + H].double()).repeat_interleave(dv, dim=1)
+        elif gate_column >= 0:
             out = out * torch.sigmoid(q[:, gate_column:gate_column + H * dv].double())
-        return out.to(q.dtype)
+        return (out * out_scale).to(q.dtype)
 
     def pair_rotate_store(self, proj, H, G, d, dv, bias, positions, freq, dims, amplitude, slots, cache, page_size, values_are_keys=False):
         """proj [T, q | k (| v)] + bias: neighbouring pairs of q (in place) and k turned, k and v (or k before it is turned)
@@ -539,11 +550,13 @@ class TorchOps:
         return out.float()
 
     def expert_rows(self, x, logits, w_gate_up, w_down, top, scale_input=False, score="sigmoid", groups=1, keep_groups=1,
-                    renormalise=False, correction=None, weight_scale=1.0, clamped=None):
+                    renormalise=False, correction=None, weight_scale=1.0, clamped=None, logit_bias=None):
         """[(token, weighted output of one of its choices)] in the order of the choices."""
         T = x.shape[0]
         E, real = logits.shape[1], w_gate_up.shape[0]
         inter = w_gate_up.shape[1] // 2
+        if logit_bias is not None:
+            logits = logits.double() + logit_bias.double()
         score = torch.softmax(logits.double(), dim=-1) if score == "softmax" else torch.sigmoid(logits.double())
         rows = []
         for t in range(T):
@@ -679,3 +692,103 @@ class TorchOps:
         part[..., 0:dims:2] = a * c - b * s
         part[..., 1:dims:2] = b * c + a * s
         out.view(T, H, out_ld)[:, :, out_col:out_col + n] = part.to(out.dtype)
+
+    # ------------------------------------------------------------------ operators of the Gepilix parts
+    @staticmethod
+    def _tanh_norm(s, norm):
+        alpha, w, b = norm
+        return torch.tanh(alpha * s) * w.double() + b.double()
+
+    def add_tanh_norm(self, x, residual, norm, scale=None, rows=None, dtype=None, members=None):
+        if members is not None:
+            outs, eps = members
+            x = sum(o.double() / torch.sqrt((o.double() ** 2).mean(-1, keepdim=True) + eps) * w.double() for o, w in outs) / len(outs)
+        s = residual.double() if residual is not None else 0.0
+        if x is not None:
+            s = s + x.double() * (scale.double() if scale is not None else 1.0)
+        dtype = dtype or x.dtype
+        if rows is not None:
+            return self._tanh_norm(s[rows.long()], norm).to(dtype), None
+        if residual is None:
+            residual = s.float()
+        else:
+            residual.copy_(s.float())
+        return self._tanh_norm(s, norm).to(dtype), residual
+
+    def linear_add_tanh_norm(self, x, w, residual, norm, scale):
+        return self.add_tanh_norm(self.linear(x, w), residual, norm, scale=scale, dtype=x.dtype)[0]
+
+    def combine_experts_tanh_norm(self, rows, shared, residual, norm, scale):
+        out = shared.double().clone() if shared is not None else torch.zeros(residual.shape, dtype=torch.float64)
+        for t, y in rows:
+            out[t] += y
+        return self.add_tanh_norm(out, residual, norm, scale=scale, dtype=self._rows_of.dtype)[0]
+
+    def linear_relu2(self, x, w):
+        return (torch.relu(self.linear(x, w).double()) ** 2).to(x.dtype)
+
+    def linear_each(self, x, w):
+        return torch.stack([self.linear(x[i], w[i]) for i in range(w.shape[0])])
+
+    def token_shift(self, h, mu, last, ctx):
+        before = torch.zeros(h.shape, dtype=torch.float64)
+        for lo, hi, slot, pos0 in self._requests(ctx):
+            before[lo + 1:hi] = h[lo:hi - 1].double()
+            before[lo] = last[slot].double() if pos0 > 0 else 0.0
+            last[slot] = h[hi - 1].float()
+        return torch.stack([h.double() + (before - h.double()) * mu[i].double() for i in range(mu.shape[0])]).to(h.dtype)
+
+    def wkv_scan(self, rkvg, z, w_bias, u, S_all, ctx, H, d):
+        T = rkvg.shape[1]
+        r, k, v = (rkvg[i].double().view(T, H, d) for i in range(3))
+        decay = torch.exp(-torch.exp(z.double() + w_bias.double())).view(T, H, d)
+        bonus = u.double().view(H, d)
+        o = torch.zeros((T, H, d), dtype=torch.float64)
+        for lo, hi, slot, pos0 in self._requests(ctx):
+            S = S_all[slot].double() if pos0 > 0 else torch.zeros((H, d, d), dtype=torch.float64)
+            for t in range(lo, hi):
+                kv = torch.einsum("hk,hv->hkv", k[t], v[t])
+                o[t] = torch.einsum("hkv,hk->hv", S + bonus[:, :, None] * kv, r[t])
+                S = decay[t][:, :, None] * S + kv
+            S_all[slot] = S.float()
+        return o.reshape(T, H * d).float()
+
+    def state_space_scan(self, xbc, dt, dt_bias, rate, D, S_all, ctx, H, G, n, dv):
+        T, inner = xbc.shape[0], H * dv
+        x = xbc[:, :inner].double().view(T, H, dv)
+        B = xbc[:, inner:inner + G * n].double().view(T, G, n).repeat_interleave(H // G, dim=1)
+        C = xbc[:, inner + G * n:].double().view(T, G, n).repeat_interleave(H // G, dim=1)
+        step = torch.nn.functional.softplus(dt.double() + dt_bias.double(), threshold=30.0)
+        decay = torch.exp(-rate.double() * step)
+        y = torch.zeros((T, H, dv), dtype=torch.float64)
+        for lo, hi, slot, pos0 in self._requests(ctx):
+            S = S_all[slot].double() if pos0 > 0 else torch.zeros((H, n, dv), dtype=torch.float64)
+            for t in range(lo, hi):
+                S = decay[t][:, None, None] * S + torch.einsum("hn,hv->hnv", B[t] * step[t][:, None], x[t])
+                y[t] = torch.einsum("hnv,hn->hv", S, C[t]) + D.double()[:, None] * x[t]
+            S_all[slot] = S.float()
+        return y.reshape(T, inner).float()
+
+    def gated_group_norm(self, y, gate, gate_column, weight, eps, groups, out, column, scale):
+        T, inner = y.shape
+        g = gate[:, gate_column:gate_column + inner].double()
+        x = (y.double() * g * torch.sigmoid(g)).view(T, groups, inner // groups)
+        x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+        out[:, column:column + inner] = (x.reshape(T, inner) * weight.double() * scale).to(out.dtype)
+
+    def gated_lru(self, u, w_gates, gate_bias, rate, yx, y_bias, S_all, ctx, out, column, scale):
+        T, n = u.shape
+        B, two_s, s = w_gates.shape
+        z = torch.einsum("tbi,boi->tbo", u.double().view(T, B, s), w_gates.double())
+        r = torch.sigmoid(z[:, :, :s].reshape(T, n) + gate_bias[0].double())
+        i = torch.sigmoid(z[:, :, s:].reshape(T, n) + gate_bias[1].double())
+        log_a = -rate.double() * r
+        a, add = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * u.double()
+        g = yx[:, :n].double() + y_bias.double()
+        g = 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3)))
+        for lo, hi, slot, pos0 in self._requests(ctx):
+            S = S_all[slot].double() if pos0 > 0 else torch.zeros(n, dtype=torch.float64)
+            for t in range(lo, hi):
+                S = a[t] * S + add[t]
+                out[t, column:column + n] = (S * g[t] * scale).to(out.dtype)
+            S_all[slot] = S.float()
