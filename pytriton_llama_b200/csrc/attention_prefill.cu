@@ -13,7 +13,9 @@
 // column gate_col + h * D of the token's q row; `pool` = P > 0 (with a window) puts key tiles of block means in front:
 // entry b of `summary` (pages laid out as the cache's, with a block table of their own) is the mean key and mean
 // value of positions bP .. bP + P - 1, seen by the query at position p if bP + P - 1 <= p - window; `sink_logits` [heads]:
-// the sink's term has that score for a head instead of 0.
+// the sink's term has that score for a head instead of 0; `softcap` = c > 0 turns a score s into c tanh(s / c); `chunk` = n > 0
+// (no window) lets the query at position p see the keys from p - p % n on; `gate_per_head`: the gate of head h is the one
+// entry at gate_col + h; `out_scale` multiplies the result.
 //
 // tiles[i] = {request row, first token index, rows (0..128; 0: nothing to do), position of the first token}.
 #include "mma_utils.cuh"
@@ -40,6 +42,9 @@ struct PrefillExtras {
   const int* sum_bt;
   int sum_bt_stride, sum_pages;
   const float* sink_logits;
+  float softcap;
+  int chunk, gate_per_head;
+  float out_scale;
 };
 
 // MT = 16-row tiles per warp: 2 for head size 64 (4 warps), 1 for 128 (8 warps).
@@ -72,7 +77,9 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
   if (rows <= 0) return;                          // an empty second half of a pair of tiles
   const int h = blockIdx.y;
   const int kvh = h / (nq / nkv);
-  const int k_lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
+  // the first position that the query at position p sees without the kept ones
+  auto low_of = [&](int p) { return window > 0 ? max(p - window + 1, 0) : (ex.chunk > 0 ? p - p % ex.chunk : 0); };
+  const int k_lo = low_of(pos0);
   const int k_end = pos0 + rows;                 // one past the last key any row of the tile sees
   // positions below `keep` stay visible when the window has passed them: those before the first window of the
   // tile come first, in key tiles of their own (no key is met twice), then the keys from k_lo on
@@ -162,6 +169,9 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
   float m_run[MT][2], l_run[MT][2];
   float row_scale[MT][2];                          // the scores' factor of a row: the scale, times the query temperature of its position
   int row_blocks[MT][2];                           // how many block means a row sees
+  const int warp_low_min = low_of(warp_qmin), warp_low_max = low_of(warp_qmax);
+  // a capped score, in the logarithm's base 2: cap2 tanh(v / cap2) = cap2 - 2 cap2 / (1 + 2^(v * 2 / cap))
+  const float cap2 = ex.softcap * 1.4426950408889634f, cap_rate = ex.softcap > 0.f ? 2.0f / ex.softcap : 0.f;
   const float slope2 = ex.bias_exp > 0.f ? exp2f(-ex.bias_exp * (float)(h + 1) / (float)nq) * 1.4426950408889634f : 0.f;
   float o[MT][D / 8][4];
 #pragma unroll
@@ -191,7 +201,7 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
     if (keep_tile && pool) {
       if (warp_qmax - window + 1 <= 0 || key_first >= (warp_qmax - window + 1) / pool) continue;   // no row of this warp sees a block of the tile
     } else if (key_first > warp_qmax) continue;                // wholly above this warp's diagonal
-    if (!keep_tile && window > 0 && key_first >= keep && key_first + kPfKeys - 1 < warp_qmin - window + 1) continue;   // wholly before its window
+    if (!keep_tile && key_first >= keep && key_first + kPfKeys - 1 < warp_low_min) continue;   // wholly before its window
     const int stage = tile % Cfg::kStages;
     const uint32_t kbase = kv_smem + stage * 2 * Cfg::kTileBytes;
     const uint32_t vbase = kbase + Cfg::kTileBytes;
@@ -217,21 +227,24 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
       }
     }
     const bool need_mask = keep_tile ? (key_first + kPfKeys > (pool ? (warp_qmin - window + 1 > 0 ? (warp_qmin - window + 1) / pool : 0) : keep_lim))
-                                     : ((key_first + kPfKeys - 1 > warp_qmin) || (window > 0 && key_first < warp_qmax - window + 1));
+                                     : ((key_first + kPfKeys - 1 > warp_qmin) || key_first < warp_low_max);
     uint32_t pa[MT][kPfKeys / 16][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const int qpos0 = pos0 + wrow0 + mt * 16 + g;
+      int row_low[2] = {0, 0};
+      if (need_mask) { row_low[0] = low_of(qpos0); row_low[1] = low_of(qpos0 + 8); }
 #pragma unroll
       for (int nt = 0; nt < kPfKeys / 8; ++nt) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           float v = s[mt][nt][e] * row_scale[mt][e >> 1];
+          if (ex.softcap > 0.f) v = cap2 - __fdividef(2.0f * cap2, 1.0f + fast_exp2(v * cap_rate));
           if (need_mask) {
             const int key = key_first + nt * 8 + 2 * c + (e & 1);
             const int qp = qpos0 + (e >> 1) * 8;
             if (keep_tile ? key >= (pool ? row_blocks[mt][e >> 1] : keep_lim)
-                          : (key > qp || (window > 0 && key < qp - window + 1 && key >= keep))) v = -INFINITY;
+                          : (key > qp || (key < row_low[e >> 1] && key >= keep))) v = -INFINITY;
           }
           if (slope2 != 0.f && !(keep_tile && pool)) {
             const int key = key_first + nt * 8 + 2 * c + (e & 1);
@@ -297,9 +310,11 @@ prefill_attention_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
 #pragma unroll
         for (int i = 0; i < D / 8; ++i) { o[mt][i][2 * hh] *= a; o[mt][i][2 * hh + 1] *= a; }
       }
-      const float inv = l_run[mt][hh] > 0.f ? 1.0f / l_run[mt][hh] : 0.f;
+      float inv = l_run[mt][hh] > 0.f ? ex.out_scale / l_run[mt][hh] : 0.f;
+      if (ex.gate_col >= 0 && ex.gate_per_head)
+        inv *= 1.0f / (1.0f + expf(-__bfloat162float(q[(size_t)(tok0 + row) * q_stride + ex.gate_col + h])));
       __nv_bfloat16* dst = out + (size_t)(tok0 + row) * out_stride + (size_t)h * D + 2 * c;
-      const __nv_bfloat16* gate = ex.gate_col >= 0 ? q + (size_t)(tok0 + row) * q_stride + ex.gate_col + (size_t)h * D + 2 * c : nullptr;
+      const __nv_bfloat16* gate = ex.gate_col >= 0 && !ex.gate_per_head ? q + (size_t)(tok0 + row) * q_stride + ex.gate_col + (size_t)h * D + 2 * c : nullptr;
 #pragma unroll
       for (int i = 0; i < D / 8; ++i) {
         float r0 = o[mt][i][2 * hh] * inv, r1 = o[mt][i][2 * hh + 1] * inv;
@@ -317,7 +332,7 @@ template <int D, int MT>
 int launch_prefill(void* out, const void* q, const void* cache, const int* block_table, const int* tiles, int n_tiles,
                    int q_stride, int out_stride, int bt_stride, int nq, int nkv, int page_size, float scale,
                    int window, int num_pages, void* stream, int keep = 0, int sink = 0, float temp_coef = 0.f, int temp_every = 1,
-                   PrefillExtras ex = {0.f, -1, 0, nullptr, nullptr, 0, 0, nullptr}) {
+                   PrefillExtras ex = {0.f, -1, 0, nullptr, nullptr, 0, 0, nullptr, 0.f, 0, 0, 1.f}) {
   using Cfg = PrefillCfg<D, MT>;
   static SmemRaised raised = {};
   if (int rc = raise_shared_memory("prefill_attention", prefill_attention_kernel<D, MT>, Cfg::kSmem, raised)) return rc;
@@ -380,14 +395,17 @@ PTL_EXPORT int ptl_prefill_attention_opts_bf16(void* out, const void* q, const v
                                                int nq, int nkv, int d, int page_size, float scale, int window, int keep,
                                                int num_pages, int sink, float temp_coef, int temp_every, float bias_exp,
                                                int gate_col, int pool, const void* summary, const int* sum_bt, int sum_bt_stride,
-                                               int sum_pages, const float* sink_logits, void* stream) {
+                                               int sum_pages, const float* sink_logits, float softcap, int chunk, int gate_per_head,
+                                               float out_scale, void* stream) {
   using namespace ptl;
   if (sink_logits) sink = 1;
   PTL_REQUIRE(pool == 0 || (summary && sum_bt && sum_pages > 0 && window > 0 && keep == 0 && !sink && aligned16(summary)),
               "prefill_attention: means of blocks need their pages and a window, and go with no kept positions or sink");
-  PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || (gate_col + nq * d <= q_stride && gate_col % 2 == 0)), "prefill_attention: bad bias or gate column");
+  PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || (gate_per_head ? gate_col + nq <= q_stride : gate_col + nq * d <= q_stride && gate_col % 2 == 0)),
+              "prefill_attention: bad bias or gate column");
+  PTL_REQUIRE(softcap >= 0.f && chunk >= 0 && (chunk == 0 || (window == 0 && keep == 0)), "prefill_attention: blocks of positions go with no window");
   const PrefillExtras ex = {bias_exp, gate_col, window > 0 ? pool : 0, (const __nv_bfloat16*)summary, sum_bt, sum_bt_stride, sum_pages,
-                            sink_logits};
+                            sink_logits, softcap, chunk, gate_per_head, out_scale};
   PTL_REQUIRE(n_tiles >= 0 && nq > 0 && nkv > 0 && page_size > 0 && num_pages > 0 && keep >= 0 && temp_every >= 1,
               "prefill_attention: bad sizes");
   PTL_REQUIRE(nq % nkv == 0, "prefill_attention: %d query heads are no multiple of %d kv heads", nq, nkv);

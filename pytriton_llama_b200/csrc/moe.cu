@@ -6,7 +6,7 @@
 //                 all experts; `groups` > 1: experts form that many groups of neighbours, a group's score is
 //                 its largest score and only experts of the `keep` best groups can be chosen (the lower group
 //                 wins a tie); `correction` [E]: experts are chosen by score + correction and weighted by the score
-//                 alone; `renorm`: the chosen scores are divided by their sum + 1e-20; `scale` multiplies the weights.
+//                 alone; `logit_bias` [E] is added to the logits first; `renorm`: the chosen scores are divided by their sum + 1e-20; `scale` multiplies the weights.
 //   moe_plan      one block: tokens per expert, each expert's rows padded to whole tiles of kMoeTile rows,
 //                 the list of tiles (expert, first row, rows), the row of every (token, choice); -1 for a choice
 //                 whose id is at or beyond the number of experts that have weights.
@@ -47,7 +47,8 @@ __device__ __forceinline__ float moe_glu(float g, float u, const GluForm& f) {
 // ------------------------------------------------------------------ route
 __global__ void __launch_bounds__(128)
 moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits, int tokens, int E,
-                 int top, int softmax, int groups, int keep, int renorm, const float* __restrict__ correction, float scale) {
+                 int top, int softmax, int groups, int keep, int renorm, const float* __restrict__ correction, float scale,
+                 const float* __restrict__ logit_bias) {
   __shared__ float s_best[4][kMoeMaxExperts];      // per warp: the largest score of every group
   pdl_wait();
   pdl_launch_dependents();
@@ -65,6 +66,7 @@ moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float
     float v = -INFINITY;
     if (e < E) {
       v = logits[(size_t)t * E + e];
+      if (logit_bias) v += logit_bias[e];
       if (!(v == v)) v = -INFINITY;        // a NaN never wins
       if (!softmax) v = sigmoid_f32(v);
     }
@@ -793,14 +795,14 @@ moe_combine_norm_kernel(float* __restrict__ residual, T* __restrict__ y, const f
 
 // ------------------------------------------------------------------ launchers
 int moe_route(int* ids, float* weights, const float* logits, int tokens, int E, int top, int softmax, int groups, int keep,
-              int renorm, const float* correction, float scale, void* stream) {
+              int renorm, const float* correction, float scale, const float* logit_bias, void* stream) {
   PTL_REQUIRE(tokens >= 0 && E >= 1 && E <= kMoeMaxExperts && top >= 1 && top <= E, "moe_route: %d experts, top %d (at most %d experts)", E, top, kMoeMaxExperts);
   PTL_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
               "moe_route: %d experts in %d groups, %d kept, top %d", E, groups, keep, top);
   PTL_REQUIRE(!correction || groups == 1, "moe_route: the correction goes with no groups");
   if (tokens == 0) return 0;
   return launch_kernel("moe_route", moe_route_kernel, dim3((tokens + 3) / 4), dim3(128), 0, as_stream(stream), ids, weights, logits,
-                       tokens, E, top, softmax, groups, keep, renorm, correction, scale);
+                       tokens, E, top, softmax, groups, keep, renorm, correction, scale, logit_bias);
 }
 
 int moe_plan(int* pos, int* tiles, int* meta, const int* ids, int n, int E, int max_tiles, int* wide, int max_wide, void* stream) {
@@ -880,8 +882,8 @@ int moe_combine_norm(float* residual, void* y, const float* C, const void* x, co
 
 PTL_EXPORT int ptl_moe_tile_rows() { return ptl::kMoeTile; }
 PTL_EXPORT int ptl_moe_route(int* ids, float* weights, const float* logits, int tokens, int E, int top, int softmax, int groups,
-                             int keep, int renorm, const float* correction, float scale, void* stream) {
-  return ptl::moe_route(ids, weights, logits, tokens, E, top, softmax, groups, keep, renorm, correction, scale, stream);
+                             int keep, int renorm, const float* correction, float scale, const float* logit_bias, void* stream) {
+  return ptl::moe_route(ids, weights, logits, tokens, E, top, softmax, groups, keep, renorm, correction, scale, logit_bias, stream);
 }
 PTL_EXPORT int ptl_moe_wide_rows() { return ptl::kMoeWide; }
 PTL_EXPORT int ptl_moe_plan(int* pos, int* tiles, int* meta, const int* ids, int n, int E, int max_tiles, int* wide, int max_wide,

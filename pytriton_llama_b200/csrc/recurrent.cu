@@ -14,14 +14,16 @@ __device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)
 
 // ------------------------------------------------------------------ causal convolution per channel
 // y[t, c] = act(b[c] + sum_k w[c, k] * in[t - (taps - 1) + k, c]), `in` being the request's inputs: rows of
-// this step, before them the taps - 1 inputs kept in the state, zeros before position 0.
+// this step (plus in_bias[c] where that is given), before them the taps - 1 inputs kept in the state (bias and all), zeros
+// before position 0.
 // state[slot, j, c], j = 0 .. taps - 2, oldest first.  Reads the state only; conv_state_kernel moves it on.
 template <typename T>
 __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x, int ld, int column, int channels,
                                    const float* __restrict__ w, const float* __restrict__ b, int taps,
                                    const float* __restrict__ state, const int* __restrict__ q_start,
                                    const int* __restrict__ tok_req, const int* __restrict__ positions,
-                                   const int* __restrict__ state_slot, int silu, float* __restrict__ state_out) {
+                                   const int* __restrict__ state_slot, int silu, float* __restrict__ state_out,
+                                   const float* __restrict__ in_bias) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
@@ -33,6 +35,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
   const int pos = positions[t];
   const float* st = state + (size_t)state_slot[r] * (taps > 1 ? taps - 1 : 1) * channels;
   float acc = b ? b[c] : 0.f;
+  const float own = in_bias ? in_bias[c] : 0.f;
   if (state_out) {
     // every request brings one token: this thread is the only one that touches its channel of the request's state, so
     // it also moves the state on (entry j takes entry j + 1, the last one the token's input)
@@ -47,7 +50,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
         v[j] = (there && pos - (taps - 1 - j) >= 0) ? st[(size_t)j * channels + c] : 0.f;
         wt[j] = there ? w[(size_t)c * taps + j] : 0.f;
       }
-      const float x_now = to_f32(x_raw);
+      const float x_now = to_f32(x_raw) + own;
 #pragma unroll
       for (int j = 0; j < kHeld; ++j) {
         if (j < taps - 1) {
@@ -60,7 +63,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
       out[(size_t)t * channels + c] = from_f32<T>(silu ? silu_f32(acc) : acc);
       return;
     }
-    const float x_now = to_f32(x_raw);
+    const float x_now = to_f32(x_raw) + own;
     for (int j = 0; j < taps - 1; ++j) {
       const float v = pos - (taps - 1 - j) >= 0 ? st[(size_t)j * channels + c] : 0.f;
       acc = fmaf(w[(size_t)c * taps + j], v, acc);
@@ -74,7 +77,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
   for (int k = 0; k < taps; ++k) {
     const int back = taps - 1 - k;
     float v = 0.f;
-    if (back <= in_step) v = to_f32(x[(size_t)(t - back) * ld + column + c]);
+    if (back <= in_step) v = to_f32(x[(size_t)(t - back) * ld + column + c]) + own;
     else if (back <= pos) v = st[(size_t)(taps - 1 - (back - in_step)) * channels + c];
     acc = fmaf(w[(size_t)c * taps + k], v, acc);
   }
@@ -87,12 +90,13 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
 template <typename T>
 __global__ void conv_state_kernel(float* __restrict__ state, const T* __restrict__ x, int ld, int column, int channels, int taps,
                                   const int* __restrict__ q_start, const int* __restrict__ positions,
-                                  const int* __restrict__ state_slot) {
+                                  const int* __restrict__ state_slot, const float* __restrict__ in_bias) {
   pdl_wait();
   pdl_launch_dependents();
   const int r = blockIdx.x;
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= channels) return;
+  const float own = in_bias ? in_bias[c] : 0.f;
   const int lo = q_start[r], n = q_start[r + 1] - lo;
   if (n <= 0 || state_slot[r] < 0) return;
   const int pos0 = positions[lo];
@@ -100,7 +104,7 @@ __global__ void conv_state_kernel(float* __restrict__ state, const T* __restrict
   for (int j = 0; j < taps - 1; ++j) {
     const int row = n - (taps - 1) + j;
     float v;
-    if (row >= 0) v = to_f32(x[(size_t)(lo + row) * ld + column + c]);
+    if (row >= 0) v = to_f32(x[(size_t)(lo + row) * ld + column + c]) + own;
     else v = pos0 + row >= 0 ? st[(size_t)(j + n) * channels + c] : 0.f;
     st[(size_t)j * channels + c] = v;
   }
@@ -413,11 +417,97 @@ gated_head_norm_kernel(T* __restrict__ out, int out_ld, int column, const float*
   }
 }
 
+// ------------------------------------------------------------------ output gate, then a norm in equal parts
+// With x = o * silu(gate):  out[t, column + e] = x[e] / sqrt(mean over e's part of x^2 + eps) * w[e] * scale, the row being cut
+// into `groups` parts of `len`.  One block per (token, part); rows of whole packets keep their x in registers (NP packets
+// of four a thread), others are worked out twice.
+template <typename T, int NP>
+__global__ void __launch_bounds__(256)
+gated_group_norm_kernel(T* __restrict__ out, int out_ld, int column, const float* __restrict__ o, int inner, const float* __restrict__ w,
+                        float eps, const T* __restrict__ gate, int gate_ld, int gate_column, int len, float scale) {
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, at = blockIdx.y * len;
+  const float* src = o + (size_t)t * inner + at;
+  const T* g = gate + (size_t)t * gate_ld + gate_column + at;
+  T* dst = out + (size_t)t * out_ld + column + at;
+  float ss = 0.f;
+  if constexpr (NP > 0) {
+    float4 x[NP];
+#pragma unroll
+    for (int n = 0; n < NP; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      x[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < len) {
+        x[n] = *reinterpret_cast<const float4*>(src + i);
+        float gv[4];
+        if constexpr (sizeof(T) == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(g + i);
+          gv[0] = v.x; gv[1] = v.y; gv[2] = v.z; gv[3] = v.w;
+        } else {
+          const uint2 raw = *reinterpret_cast<const uint2*>(g + i);
+          const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+          const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+          gv[0] = a.x; gv[1] = a.y; gv[2] = b.x; gv[3] = b.y;
+        }
+        x[n].x *= silu_f32(gv[0]); x[n].y *= silu_f32(gv[1]); x[n].z *= silu_f32(gv[2]); x[n].w *= silu_f32(gv[3]);
+        ss = fmaf(x[n].x, x[n].x, fmaf(x[n].y, x[n].y, fmaf(x[n].z, x[n].z, fmaf(x[n].w, x[n].w, ss))));
+      }
+    }
+    const float f = scale / sqrtf(block_sum(ss, red) / (float)len + eps);
+#pragma unroll
+    for (int n = 0; n < NP; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i >= len) continue;
+      const float4 wv = *reinterpret_cast<const float4*>(w + at + i);
+      const float4 y = make_float4(x[n].x * f * wv.x, x[n].y * f * wv.y, x[n].z * f * wv.z, x[n].w * f * wv.w);
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(dst + i) = y;
+      } else {
+        uint2 raw;
+        *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(y.x, y.y);
+        *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(y.z, y.w);
+        *reinterpret_cast<uint2*>(dst + i) = raw;
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < len; i += 256) {
+      const float x = src[i] * silu_f32(to_f32(g[i]));
+      ss = fmaf(x, x, ss);
+    }
+    const float f = scale / sqrtf(block_sum(ss, red) / (float)len + eps);
+    for (int i = threadIdx.x; i < len; i += 256) dst[i] = from_f32<T>(src[i] * silu_f32(to_f32(g[i])) * f * w[at + i]);
+  }
+}
+
 // ------------------------------------------------------------------ launchers
+template <typename T>
+int gated_group_norm(void* out, int out_ld, int column, const float* o, const float* w, float eps, const void* gate, int gate_ld,
+                     int gate_column, int tokens, int inner, int groups, float scale, void* stream) {
+  PTL_REQUIRE(tokens >= 0 && inner > 0 && groups > 0 && groups <= 65535 && inner % groups == 0 && eps > 0.f && column >= 0 &&
+              column + inner <= out_ld && gate_column >= 0 && gate_column + inner <= gate_ld,
+              "gated_group_norm: bad sizes tokens=%d inner=%d groups=%d", tokens, inner, groups);
+  if (tokens == 0) return 0;
+  const int len = inner / groups;
+  const T* g = (const T*)gate + gate_column;
+  T* dst = (T*)out + column;
+  const bool vec = len % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && aligned16(o) && aligned16(w) &&
+                   ((uintptr_t)g % (4 * sizeof(T))) == 0 && ((uintptr_t)dst % (4 * sizeof(T))) == 0;
+#define PTL_GGN(NP) return launch_kernel("gated_group_norm", gated_group_norm_kernel<T, NP>, dim3(tokens, groups), dim3(256), 0, \
+    as_stream(stream), (T*)out, out_ld, column, o, inner, w, eps, (const T*)gate, gate_ld, gate_column, len, scale)
+  if (vec && len <= 1024) PTL_GGN(1);
+  if (vec && len <= 2048) PTL_GGN(2);
+  if (vec && len <= 4096) PTL_GGN(4);
+  if (vec && len <= 8192) PTL_GGN(8);
+  PTL_GGN(0);
+#undef PTL_GGN
+}
+
 template <typename T>
 int causal_conv(void* out, const void* x, int ld, int column, int channels, const float* w, const float* b, int taps, float* state,
                 const int* q_start, const int* tok_req, const int* positions, const int* state_slot, int tokens, int requests,
-                int silu, int single_tokens, void* stream) {
+                int silu, int single_tokens, const float* in_bias, void* stream) {
   PTL_REQUIRE(tokens >= 0 && requests >= 0 && channels > 0 && taps > 0 && column >= 0 && column + channels <= ld,
               "causal_conv: bad sizes tokens=%d channels=%d taps=%d column=%d ld=%d", tokens, channels, taps, column, ld);
   if (tokens == 0) return 0;
@@ -427,11 +517,11 @@ int causal_conv(void* out, const void* x, int ld, int column, int channels, cons
   float* state_out = (single_tokens && taps > 1) ? state : nullptr;
   if (int rc = launch_kernel("causal_conv", causal_conv_kernel<T>, dim3(tokens, tiles.x), block, 0, as_stream(stream), (T*)out,
                              (const T*)x, ld, column, channels, w, b, taps, (const float*)state, q_start, tok_req, positions,
-                             state_slot, silu, state_out))
+                             state_slot, silu, state_out, in_bias))
     return rc;
   if (taps == 1 || requests == 0 || state_out) return 0;
   return launch_kernel("conv_state", conv_state_kernel<T>, dim3(requests, tiles.x), block, 0, as_stream(stream), state, (const T*)x,
-                       ld, column, channels, taps, q_start, positions, state_slot);
+                       ld, column, channels, taps, q_start, positions, state_slot, in_bias);
 }
 
 template <typename T>
@@ -500,9 +590,9 @@ int gated_head_norm(void* out, int out_ld, int column, const float* o, const flo
   PTL_EXPORT int ptl_causal_conv##SUFFIX(void* out, const void* x, int ld, int column, int channels, const float* w,               \
                                          const float* b, int taps, float* state, const int* q_start, const int* tok_req,           \
                                          const int* positions, const int* state_slot, int tokens, int requests, int silu,         \
-                                         int single_tokens, void* stream) {                                                       \
+                                         int single_tokens, const float* in_bias, void* stream) {                                 \
     return ptl::causal_conv<TYPE>(out, x, ld, column, channels, w, b, taps, state, q_start, tok_req, positions, state_slot, tokens, \
-                                  requests, silu, single_tokens, stream);                                                         \
+                                  requests, silu, single_tokens, in_bias, stream);                                                \
   }                                                                                                                               \
   PTL_EXPORT int ptl_selective_scan##SUFFIX(void* out, const void* xc, const float* dt_raw, const float* dt_bias, const float* A,  \
                                             const void* bc, const float* D, const void* z, int z_ld, int z_column, int inner,      \
@@ -524,5 +614,14 @@ int gated_head_norm(void* out, int out_ld, int column, const float* o, const flo
     return ptl::gated_head_norm<TYPE>(out, out_ld, column, o, w, eps, gate, gate_ld, gate_column, tokens, heads, dv, scale,        \
                                       sigmoid_gate, weight_per_head, stream);                                                     \
   }
+#define PTL_GATED_GROUP_NORM(SUFFIX, TYPE)                                                                                        \
+  PTL_EXPORT int ptl_gated_group_norm##SUFFIX(void* out, int out_ld, int column, const float* o, const float* w, float eps,        \
+                                              const void* gate, int gate_ld, int gate_column, int tokens, int inner, int groups,  \
+                                              float scale, void* stream) {                                                        \
+    return ptl::gated_group_norm<TYPE>(out, out_ld, column, o, w, eps, gate, gate_ld, gate_column, tokens, inner, groups, scale,   \
+                                       stream);                                                                                   \
+  }
+PTL_GATED_GROUP_NORM(_f32, float)
+PTL_GATED_GROUP_NORM(_bf16, __nv_bfloat16)
 PTL_RECURRENT(_f32, float)
 PTL_RECURRENT(_bf16, __nv_bfloat16)

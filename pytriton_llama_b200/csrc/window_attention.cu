@@ -27,7 +27,9 @@
 // sigmoid of the dv entries at column gate_col + h * dv of the token's q row.  `pool` = P > 0 (with a window): the list
 // starts with one mean key and mean value for every block b of P positions with bP + P - 1 <= p - window, read from
 // `summary`, pages of the cache's layout with a block table of their own; that part of the list is padded to whole
-// turns of 32 so that a turn reads either means or tokens.
+// turns of 32 so that a turn reads either means or tokens.  `softcap` = c > 0: a score s becomes c tanh(s / c).  `chunk` = n > 0
+// (no window): the visible keys are those from p - p % n on.  `gate_per_head`: the gate of head h is the one entry at
+// gate_col + h.  `out_scale` multiplies the result.
 //
 // head_norm_rotate_store, per token, on [T, q | k | v | ...]: every q and k head divided by its own root mean square
 // and multiplied by the weight [d] of its kind (eps > 0), entries i and i + rot/2 of a head turned by
@@ -405,6 +407,19 @@ int pool_blocks(void* summary, const void* cache, const int* block_table, const 
 constexpr int kWaMaxPerLane = 16;  // value heads up to 512 (kernels are built for 8 and for 16 values per lane)
 constexpr int kWaWarps = 4;
 
+struct WaExtras {
+  float softcap;
+  int chunk, gate_per_head;
+  float out_scale;
+};
+// The factor of entry dd of head h: the result's scale, and the gate where there is one.
+template <typename T>
+__device__ __forceinline__ float wa_factor(const T* __restrict__ gate_row, int h, int dv, int dd, const WaExtras& ex) {
+  if (!gate_row) return ex.out_scale;
+  const float g = to_f32(gate_row[ex.gate_per_head ? h : h * dv + dd]);
+  return ex.out_scale / (1.0f + expf(-g));
+}
+
 __device__ __forceinline__ void wa_two_fma(float& hi, float& lo, float a, float b) {
   const float h = __fmul_rn(a, b);
   const float r = fmaf(a, b, -h);
@@ -432,7 +447,7 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
                         int splits, int num_pages, int vec_ok, const int* __restrict__ items, int wide_ok, int shared_v,
                         int sink, float temp_coef, int temp_every, float bias_exp, int gate_col, int pool,
                         const T* __restrict__ summary, const int* __restrict__ sum_bt, int sum_bt_stride, int sum_pages,
-                        const float* __restrict__ sink_logits) {
+                        const float* __restrict__ sink_logits, const WaExtras ex) {
   constexpr int kWaMaxPerLane = MPL;   // values of a head that a lane holds
   extern __shared__ float qs_all[];  // [warps][d]
   __shared__ float s_pr[kWaWarps][32];
@@ -453,7 +468,7 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
   for (int i = lane; i < d; i += 32) qs[i] = kCompensated ? to_f32(qrow[i]) : to_f32(qrow[i]) * scale;
   __syncwarp();
 
-  const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+  const int lo = ex.chunk > 0 ? p - p % ex.chunk : (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
   const int n_keep = min(keep, lo);                 // kept positions that the window has passed
   const int n_pool = (pool > 0 && window > 0 && r >= 0 && p - window + 1 > 0) ? (p - window + 1) / pool : 0;   // whole blocks behind the window
   const int n_pool_pad = (n_pool + 31) & ~31;
@@ -519,6 +534,7 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
         }
       }
       s = kCompensated ? __fadd_rn(dot, dot_lo) * scale : dot;
+      if (ex.softcap > 0.f) s = ex.softcap * tanhf(s / ex.softcap);
       if (!mean) s = fmaf(-slope, (float)(p - key), s);
     }
     const float m_new = fmaxf(m, warp_max(s));
@@ -615,15 +631,11 @@ window_attention_kernel(T* __restrict__ out, float* __restrict__ part_acc, float
     }
     const float inv = l > 0.f ? 1.0f / l : 0.f;
     T* o = out + (size_t)t * out_stride + (size_t)h * dv;
-    const T* gate = gate_col >= 0 ? q + (size_t)t * q_stride + gate_col + (size_t)h * dv : nullptr;
+    const T* gate = gate_col >= 0 ? q + (size_t)t * q_stride + gate_col : nullptr;
 #pragma unroll
     for (int i = 0; i < kWaMaxPerLane; ++i) {
       const int dd = wide_ok ? lane * wide_ok + i : lane + 32 * i;
-      if (dd < dv && (!wide_ok || i < wide_ok)) {
-        float res = acc[i] * inv;
-        if (gate) res *= 1.0f / (1.0f + expf(-to_f32(gate[dd])));
-        o[dd] = from_f32<T>(res);
-      }
+      if (dd < dv && (!wide_ok || i < wide_ok)) o[dd] = from_f32<T>(acc[i] * inv * wa_factor(gate, h, dv, dd, ex));
     }
   } else {
     const size_t idx = ((size_t)t * H + h) * splits + split;
@@ -642,7 +654,8 @@ template <typename T, int MPL>
 __global__ void __launch_bounds__(kWaWarps * 32)
 window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                               int out_stride, int H, int dv, int splits, int tokens, const int* __restrict__ items, int sink,
-                              const T* __restrict__ q, int q_stride, int gate_col, const float* __restrict__ sink_logits) {
+                              const T* __restrict__ q, int q_stride, int gate_col, const float* __restrict__ sink_logits,
+                              const WaExtras ex) {
   constexpr int kWaMaxPerLane = MPL;
   pdl_wait();
   pdl_launch_dependents();
@@ -702,15 +715,11 @@ window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ par
   if (sink) L += expf(z_sink - M);
   const float inv = L > 0.f ? 1.0f / L : 0.f;
   T* o = out + (size_t)t * out_stride + (size_t)h * dv;
-  const T* gate = gate_col >= 0 ? q + (size_t)t * q_stride + gate_col + (size_t)h * dv : nullptr;
+  const T* gate = gate_col >= 0 ? q + (size_t)t * q_stride + gate_col : nullptr;
 #pragma unroll
   for (int i = 0; i < kWaMaxPerLane; ++i) {
     const int dd = lane + 32 * i;
-    if (dd < dv) {
-      float res = acc[i] * inv;
-      if (gate) res *= 1.0f / (1.0f + expf(-to_f32(gate[dd])));
-      o[dd] = from_f32<T>(res);
-    }
+    if (dd < dv) o[dd] = from_f32<T>(acc[i] * inv * wa_factor(gate, h, dv, dd, ex));
   }
 }
 
@@ -720,12 +729,15 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                      int bt_stride, int H, int G, int d, int dv, int page_size, float scale, int window, int keep, int splits,
                      int num_pages, const int* items, int shared_v, int sink, float temp_coef, int temp_every, float bias_exp,
                      int gate_col, int pool, const void* summary, const int* sum_bt, int sum_bt_stride, int sum_pages,
-                     const float* sink_logits, void* stream) {
+                     const float* sink_logits, const WaExtras& ex, void* stream) {
   PTL_REQUIRE(tokens >= 0 && H > 0 && G > 0 && page_size > 0 && d > 0, "window_attention: bad sizes");
   if (sink_logits) sink = 1;
   PTL_REQUIRE(pool == 0 || (summary && sum_bt && sum_pages > 0 && window > 0 && keep == 0 && !shared_v && !sink),
               "window_attention: means of blocks need their pages and a window, and go with no kept positions, shared values or sink");
-  PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || gate_col + H * dv <= q_stride), "window_attention: bad bias or gate column");
+  PTL_REQUIRE(bias_exp >= 0.f && (gate_col < 0 || gate_col + (ex.gate_per_head ? H : H * dv) <= q_stride),
+              "window_attention: bad bias or gate column");
+  PTL_REQUIRE(ex.softcap >= 0.f && ex.chunk >= 0 && (ex.chunk == 0 || (window == 0 && keep == 0)),
+              "window_attention: blocks of positions go with no window");
   PTL_REQUIRE(!shared_v || dv <= d, "window_attention: values of %d entries inside keys of %d", dv, d);
   PTL_REQUIRE(temp_every >= 1, "window_attention: temp_every=%d", temp_every);
   PTL_REQUIRE(H % G == 0, "window_attention: %d query heads are no multiple of %d kv heads", H, G);
@@ -753,12 +765,12 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                            as_stream(stream), (T*)out, part_acc, part_ml, (const T*)q, (const T*)cache, block_table, tok_req,      \
                            positions, q_stride, out_stride, bt_stride, H, G, d, dv, page_size, scale, window, keep, splits,        \
                            num_pages, vec_ok, items, wide_ok, shared_v, sink, temp_coef, temp_every, bias_exp, gate_col, pool,     \
-                           (const T*)summary, sum_bt, sum_bt_stride, sum_pages, sink_logits);                                     \
+                           (const T*)summary, sum_bt, sum_bt_stride, sum_pages, sink_logits, ex);                                 \
     if (rc || splits <= 1) return rc;                                                                                              \
     return launch_kernel("window_attention_merge", window_attention_merge_kernel<T, MPL>,                                          \
                          dim3((unsigned)((pairs + kWaWarps - 1) / kWaWarps)), dim3(kWaWarps * 32), 0, as_stream(stream), (T*)out,  \
                          (const float*)part_acc, (const float*)part_ml, out_stride, H, dv, splits, tokens, items, sink,            \
-                         (const T*)q, q_stride, gate_col, sink_logits);                                                            \
+                         (const T*)q, q_stride, gate_col, sink_logits, ex);                                                        \
   }
   if (dv <= 32 * 8) PTL_WA_LAUNCH(8)      // (value heads up to 256 keep the registers of 8 values per lane)
   PTL_WA_LAUNCH(16)
@@ -781,11 +793,13 @@ int window_attention(void* out, const void* q, const void* cache, const int* blo
                                               int page_size, float scale, int window, int keep, int splits, int num_pages,         \
                                               const int* items, int shared_v, int sink, float temp_coef, int temp_every,           \
                                               float bias_exp, int gate_col, int pool, const void* summary, const int* sum_bt,      \
-                                              int sum_bt_stride, int sum_pages, const float* sink_logits, void* stream) {          \
+                                              int sum_bt_stride, int sum_pages, const float* sink_logits, float softcap,           \
+                                              int chunk, int gate_per_head, float out_scale, void* stream) {                       \
     return ptl::window_attention<TYPE>(out, q, cache, block_table, tok_req, positions, part_acc, part_ml, tokens, q_stride,        \
                                        out_stride, bt_stride, H, G, d, dv, page_size, scale, window, keep, splits, num_pages,      \
                                        items, shared_v, sink, temp_coef, temp_every, bias_exp, gate_col, pool, summary, sum_bt,    \
-                                       sum_bt_stride, sum_pages, sink_logits, stream);                                             \
+                                       sum_bt_stride, sum_pages, sink_logits, ptl::WaExtras{softcap, chunk, gate_per_head, out_scale}, \
+                                       stream);                                                                                    \
   }                                                                                                                                \
   PTL_EXPORT int ptl_head_norm_rotate_store##SUFFIX(void* proj, int tokens, int ld, int H, int G, int d, int dv, const float* wq,   \
                                                     const float* wk, float eps, const int* positions, const void* inv_freq,        \

@@ -35,7 +35,7 @@ _SIGNATURES = {
     "ptl_clamped_glu": [_ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _c_f, _c_f, _ptr],
     "ptl_token_side": [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr],
     "ptl_causal_conv": [_ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int,
-                        _c_int, _c_int, _ptr],
+                        _c_int, _c_int, _ptr, _ptr],
     "ptl_selective_scan": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _ptr,
                            _c_int, _ptr],
     "ptl_gated_delta_rule": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f,
@@ -51,7 +51,7 @@ _SIGNATURES = {
                                  _ptr, _c_int, _c_ll, _ptr],
     "ptl_window_attention": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                              _c_int, _c_int, _c_f, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _c_int, _c_f, _c_int, _c_f, _c_int,
-                             _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr],
+                             _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _c_f, _c_int, _c_int, _c_f, _ptr],
     "ptl_pair_rotate_store": [_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr, _c_int, _c_ll,
                               _ptr],
     "ptl_head_norm_rotate_store": [_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _ptr, _c_f, _ptr, _ptr, _c_int, _c_int,
@@ -72,6 +72,15 @@ _SIGNATURES = {
     "ptl_head_linear": [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr],
     "ptl_gla_scan": [_ptr, _ptr, _c_int, _ptr, _ptr, _c_f, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr, _c_f,
                      _ptr],
+    "ptl_wkv_scan": [_ptr, _ptr, _c_ll, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr],
+    "ptl_state_space_scan": [_ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr],
+    "ptl_gated_group_norm": [_ptr, _c_int, _c_int, _ptr, _ptr, _c_f, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr],
+    "ptl_gated_lru_scan": [_ptr, _c_int, _c_int, _ptr, _ptr, _c_ll, _c_ll, _c_int, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr,
+                           _c_int, _c_int, _c_int, _c_f, _ptr],
+    "ptl_token_shift": [_ptr, _c_ll, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr],
+    "ptl_relu2": [_ptr, _c_ll, _ptr],
+    "ptl_add_tanh_norm": [_ptr, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _c_f, _ptr, _c_int, _c_int, _ptr, _ptr, _ptr, _c_int, _c_f,
+                          _ptr, _ptr, _ptr, _c_int, _ptr],
     "ptl_moe_gather": [_ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr],
     "ptl_moe_grouped": [_ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_f, _c_f, _ptr],
     "ptl_moe_combine_norm": [_ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_f, _ptr],
@@ -182,11 +191,11 @@ def load_library() -> ctypes.CDLL:
     lib.ptl_softcap.restype = _c_int
     lib.ptl_prefill_attention_opts_bf16.argtypes = [_ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                                     _c_int, _c_int, _c_f, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_f, _c_int,
-                                                    _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _ptr]
+                                                    _c_int, _ptr, _ptr, _c_int, _c_int, _ptr, _c_f, _c_int, _c_int, _c_f, _ptr]
     lib.ptl_prefill_attention_opts_bf16.restype = _c_int
     lib.ptl_moe_tile_rows.argtypes = []
     lib.ptl_moe_tile_rows.restype = _c_int
-    lib.ptl_moe_route.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _c_f, _ptr]
+    lib.ptl_moe_route.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _c_f, _ptr, _ptr]
     lib.ptl_moe_route.restype = _c_int
     lib.ptl_moe_plan.argtypes = [_ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr]
     lib.ptl_moe_plan.restype = _c_int
@@ -200,6 +209,9 @@ def load_library() -> ctypes.CDLL:
     lib.ptl_lowrank_tanh_linear.restype = _c_int
     lib.ptl_head_linear_few_bf16.argtypes = _SIGNATURES["ptl_head_linear"]
     lib.ptl_head_linear_few_bf16.restype = _c_int
+    lib.ptl_gated_lru_single_bf16.argtypes = [_ptr, _c_int, _c_int, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr,
+                                              _ptr, _c_int, _c_int, _c_f, _ptr]
+    lib.ptl_gated_lru_single_bf16.restype = _c_int
     lib.ptl_last_error.restype = ctypes.c_char_p
     lib.ptl_set_dependent_launch.argtypes = [_c_int]
     lib.ptl_get_dependent_launch.restype = _c_int
@@ -306,6 +318,9 @@ class CudaOps:
         "add_layernorm": "norm", "xielu": "elementwise", "lowrank_tanh_linear": "recurrent", "general_delta_scan": "recurrent",
         "latent_norm_store": "rope", "rotate_head_part": "rope", "head_linear": "product",
         "latent_gather": "attention", "causal_softmax_rows": "attention",
+        "add_tanh_norm": "norm", "linear_add_tanh_norm": "product", "combine_experts_tanh_norm": "experts", "linear_relu2": "product",
+        "linear_each": "product", "token_shift": "elementwise", "wkv_scan": "recurrent", "state_space_scan": "recurrent",
+        "gated_group_norm": "norm", "gated_lru": "recurrent",
         "head_norm_rotate_store": "rope", "pool_blocks": "attention", "post_norm_add": "norm", "mean_of_normed": "norm",
     }
 
@@ -589,6 +604,11 @@ class CudaOps:
             ld = out.shape[1]
         elif epi == self.EPI_F32 and M > 64 and splits > 1:
             out = self.empty((splits, M, N), torch.float32)      # partial sums of the parts of the K range
+            ld = N
+        elif out is not None and epi == self.EPI_BF16:
+            self._want(out, "out", torch.bfloat16)
+            if tuple(out.shape) != (M, N):
+                raise KernelError("gemm_tc: the result's place does not fit")
             ld = N
         else:
             out = self.empty((M, N), torch.float32 if epi == self.EPI_F32 else torch.bfloat16)
@@ -1048,14 +1068,15 @@ class CudaOps:
                        _p(w_gate), _p(w_proj), _p(norm_w), residual.shape[0], residual.shape[1], float(eps), self._stream()))
 
     def causal_conv(self, x: torch.Tensor, column: int, channels: int, w: torch.Tensor, b: Optional[torch.Tensor],
-                    state: torch.Tensor, ctx, silu: bool = True) -> torch.Tensor:
-        """Causal convolution per channel over columns ``column``.. of x [T, ld] with the taps w [channels, taps] (the last
+                    state: torch.Tensor, ctx, silu: bool = True, in_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Causal convolution per channel over columns ``column``.. of x [T, ld] (+ ``in_bias``) with the taps w [channels, taps] (the last
         is the current token's); ``state`` [slots, taps - 1, channels] holds each request's last inputs and is moved on."""
         self._want(x, "x")
         self._want(w, "conv weight", torch.float32)
         self._want(state, "conv state", torch.float32)
-        if b is not None:
-            self._want(b, "conv bias", torch.float32)
+        for name, t in (("conv bias", b), ("conv input bias", in_bias)):
+            if t is not None:
+                self._want(t, name, torch.float32)
         taps = w.shape[1]
         if w.shape[0] != channels or state.shape[1] != max(taps - 1, 1) or state.shape[2] != channels:
             raise KernelError(f"causal_conv: weight {list(w.shape)} and state {list(state.shape)} do not fit {channels} channels")
@@ -1066,7 +1087,7 @@ class CudaOps:
         fn = getattr(self.lib, "ptl_causal_conv" + _suffix(x.dtype))
         self._check(fn(_p(out), _p(x), x.shape[1], int(column), int(channels), _p(w), _p(b), taps, _p(state), _p(ctx.q_start),
                        _p(ctx.tok_req), _p(ctx.positions), _p(ctx.state_slot), x.shape[0], ctx.num_requests, int(bool(silu)),
-                       single, self._stream()), kernels=2 if taps > 1 and not single else 1)
+                       single, _p(in_bias), self._stream()), kernels=2 if taps > 1 and not single else 1)
         return out
 
     def selective_scan(self, xc: torch.Tensor, dt: torch.Tensor, dt_b: torch.Tensor, A: torch.Tensor, bc: torch.Tensor,
@@ -1231,7 +1252,8 @@ class CudaOps:
                          temp_every: int = 1, shared_values: bool = False, distance_bias: float = 0.0, gate_column: int = -1,
                          pool: int = 0, summary: Optional[torch.Tensor] = None,
                          summary_table: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-                         column: int = 0) -> torch.Tensor:
+                         column: int = 0, softcap: float = 0.0, chunk: int = 0, gate_per_head: bool = False,
+                         out_scale: float = 1.0) -> torch.Tensor:
         """Softmax attention of every token over the keys j <= p of its request with p - j < window or j < keep_first
         (window 0: all); q is [T, >= H*d], the result [T, H*dv], or columns ``column``.. of ``out``.  ``sink``: one more
         term in the denominator, of score 0 (True) or of the head's own score (float32 [H]); ``temp_coef``: scores of the query at position p times 1 + temp_coef * ln(floor((p + 1) /
@@ -1239,7 +1261,9 @@ class CudaOps:
         ``distance_bias`` = c: head h takes 2^(-c (h + 1) / H) * (p - j) off its scores; ``gate_column``: the heads are
         multiplied by the sigmoid of q's columns from there; ``pool`` = P with ``summary`` (pages of mean keys and
         values, laid out as the cache's) and its block table: every block of P positions that lies wholly behind the
-        window is seen as its mean."""
+        window is seen as its mean.  ``softcap`` = c: a score s becomes c tanh(s / c); ``chunk`` = n (no window): only keys of
+        the query's own block of n positions are seen; ``gate_per_head``: the gate is one column per head; ``out_scale``
+        multiplies the result."""
         self._want(q, "q")
         self._want(cache, "cache", q.dtype)
         for name, t in (("block_table", block_table), ("tok_req", tok_req), ("positions", positions)):
@@ -1269,7 +1293,7 @@ class CudaOps:
         else:
             pooled = (0, None, None, 0, 0)
         options = (int(bool(shared_values)), int(bool(sink)), float(temp_coef), int(temp_every), float(distance_bias),
-                   int(gate_column), *pooled, _p(sink_logits))
+                   int(gate_column), *pooled, _p(sink_logits), float(softcap), int(chunk), int(bool(gate_per_head)), float(out_scale))
         aligned = out.data_ptr() % 16 == 0 and out.stride(0) % 2 == 0
         if (aligned and q.dtype == torch.bfloat16 and d == dv and d in (64, 128) and not shared_values and self._work(hints, "prefill_tiles") is not None
                 and self._work(hints, "decode_items") is not None and os.environ.get("PTL_WINDOW_TC", "1") != "0"):
@@ -1279,10 +1303,14 @@ class CudaOps:
         longest = getattr(hints, "max_ctx_len", 0) or block_table.shape[1] * page_size
         if window:
             longest = min(longest, window + keep_first + (longest // pooled[0] + 32 if pooled[0] else 0))
+        elif chunk:
+            longest = min(longest, chunk)
         splits = self._window_splits(tokens, H, longest)
         self._window_attention_simt(out, q, cache, block_table, tok_req, positions, H, G, d, dv, page_size, scale, window,
                                     keep_first, splits, None, options)
         return whole
+
+    WINDOW_OPTIONS = (0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0, None, 0.0, 0, 0, 1.0)      # the options at rest
 
     def _window_splits(self, tokens: int, H: int, longest: int) -> int:
         """Parts of a token's key list for the CUDA-core kernel: enough warps to fill the SMs, at least 64 keys each."""
@@ -1293,8 +1321,9 @@ class CudaOps:
                                keep_first, splits, rows, options=(0, 0, 0.0, 1)) -> None:
         """``rows``: None for every token row, else (int32 row indices or None for 0..n-1, n).  ``options``: (values
         inside the keys, sink term, temperature coefficient, temperature step[, distance bias exponent, gate column,
-        block length of the means, their pages, their block table, its width, number of their pages[, sink scores]])."""
-        options = (*options, *(0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0, None)[len(options):])
+        block length of the means, their pages, their block table, its width, number of their pages[, sink scores[, score
+        cap, block of positions, one gate per head, factor of the result]]])."""
+        options = (*options, *self.WINDOW_OPTIONS[len(options):])
         tokens = q.shape[0]
         items, n_rows = (None, tokens) if rows is None else rows
         part_acc = part_ml = None
@@ -1308,10 +1337,11 @@ class CudaOps:
                     kernels=2 if splits > 1 else 1)
 
     def _window_attention_tensor_cores(self, out, q, cache, block_table, tok_req, positions, H, G, d, page_size, scale, window,
-                                       keep_first, hints, options=(0, 0, 0.0, 1, 0.0, -1, 0, None, None, 0, 0, None)) -> bool:
+                                       keep_first, hints, options=WINDOW_OPTIONS) -> bool:
         """bfloat16, key and value heads of 64 or 128: the portions of a step on the tensor cores (the warp-level prompt
         kernel, which walks the kept first keys as key tiles of their own before the window's), its single tokens on
         the CUDA-core kernel with their key lists split; both write their rows of ``out``."""
+        options = (*options, *self.WINDOW_OPTIONS[len(options):])
         dec, tiles = hints.work["decode_items"], hints.work["prefill_tiles"]
         if tiles.items:
             rc = self.lib.ptl_prefill_attention_opts_bf16(
@@ -1323,7 +1353,9 @@ class CudaOps:
         if dec.items:
             longest = getattr(hints, "max_ctx_len", 0) or block_table.shape[1] * page_size
             if window:
-                longest = min(longest, window + keep_first + (longest // options[6] + 32 if len(options) > 6 and options[6] else 0))
+                longest = min(longest, window + keep_first + (longest // options[6] + 32 if options[6] else 0))
+            elif options[13]:
+                longest = min(longest, options[13])
             self._window_attention_simt(out, q, cache, block_table, tok_req, positions, H, G, d, d, page_size, scale, window,
                                         keep_first, self._window_splits(dec.items, H, longest),
                                         (None if dec.in_order else dec.tensor, dec.items), options)
@@ -1715,11 +1747,11 @@ class CudaOps:
     def expert_rows(self, x: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, top: int,
                     scale_input: bool = False, score: str = "sigmoid", groups: int = 1, keep_groups: int = 1,
                     renormalise: bool = False, correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
-                    clamped: Optional[Tuple[float, float, float]] = None) -> "ExpertRows":
+                    clamped: Optional[Tuple[float, float, float]] = None, logit_bias: Optional[torch.Tensor] = None) -> "ExpertRows":
         """Everything of ``routed_experts`` up to the experts' outputs, which lie sorted by expert.  ``score`` "softmax": the
         scores are the softmax over all experts; ``groups`` > 1: only experts of the ``keep_groups`` groups of neighbours
         with the largest best score can be chosen; ``correction`` float32 [E]: experts are chosen by score + correction and
-        weighted by the score; ``renormalise``: chosen scores divided by their sum; ``weight_scale`` multiplies the weights.
+        weighted by the score; ``logit_bias`` float32 [E] is added to the logits; ``renormalise``: chosen scores divided by their sum; ``weight_scale`` multiplies the weights.
         Logits beyond the experts that have weights belong to experts that hand their input on (they get no row).
         ``clamped`` = (limit, alpha, shift): an expert's inner value is min(g, limit) * sigmoid(alpha * min(g, limit)) *
         (clamp(u, +-limit) + shift) instead of silu(g) * u."""
@@ -1739,6 +1771,10 @@ class CudaOps:
             self._want(correction, "correction", torch.float32)
             if correction.numel() != E_all:
                 raise KernelError("expert_rows: one correction per expert")
+        if logit_bias is not None:
+            self._want(logit_bias, "logit bias", torch.float32)
+            if logit_bias.numel() != E_all:
+                raise KernelError("expert_rows: one logit bias per expert")
         if score not in ("sigmoid", "softmax"):
             raise KernelError(f"expert_rows: score {score!r}")
         n = T * top
@@ -1755,7 +1791,7 @@ class CudaOps:
         weights = self.empty((n,), torch.float32)
         self._check(self.lib.ptl_moe_route(_p(ids), _p(weights), _p(logits), T, E_all, top, int(score == "softmax"), int(groups),
                                            int(keep_groups) if groups > 1 else 1, int(bool(renormalise)), _p(correction),
-                                           float(weight_scale), stream))
+                                           float(weight_scale), _p(logit_bias), stream))
         self._check(self.lib.ptl_moe_plan(_p(pos), _p(tiles), _p(meta), _p(ids), n, E, max_tiles, _p(wide), max_wide, stream))
         rows = max_tiles * tile
         sorted_x = self.empty((rows, width), x.dtype)
@@ -1802,6 +1838,198 @@ class CudaOps:
         self._check(fn(_p(residual), _p(y), _p(rows.y), _p(x), _p(add), _p(shared), _p(rows.pos), _p(rows.weights), _p(weight), T, rows.top,
                        width, float(eps), self._stream()))
         return y
+
+    # ------------------------------------------------------------------ operators of the Gepilix parts
+    def add_tanh_norm(self, x: Optional[torch.Tensor], residual: Optional[torch.Tensor], norm, scale: Optional[torch.Tensor] = None,
+                      rows: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None, members=None, experts=None):
+        """(y, residual): residual (float32, in place; created when None) += scale * o and y = tanh(alpha * residual) * w + b for
+        ``norm`` = (alpha, w, b).  o is ``x`` (of y's type or float32), or with ``members`` = ([(x_m, w_m)], eps) the mean of the
+        x_m / rms(x_m) * w_m, or with ``experts`` (an ``ExpertRows``) the weighted sum of the chosen experts' outputs + ``x``.
+        With ``rows`` (int32 indices) only those rows are worked and no residual is written."""
+        alpha, w, b = norm
+        a1 = w0 = w1 = None
+        eps, count = 0.0, 0
+        if members is not None:
+            outs, eps = members
+            count = len(outs)
+            if x is not None or not 1 <= count <= 2:
+                raise KernelError("add_tanh_norm: one or two members and no other output")
+            x, w0 = outs[0]
+            if count > 1:
+                a1, w1 = outs[1]
+                self._want(a1, "second member", x.dtype)
+                if a1.shape != x.shape:
+                    raise KernelError("add_tanh_norm: the members differ in shape")
+            for t in (w0, w1):
+                if t is not None:
+                    self._want(t, "member weight", torch.float32)
+        src = x if x is not None else residual
+        width = w.numel()
+        dtype = dtype or src.dtype
+        for name, t in (("norm weight", w), ("norm bias", b), ("scale", scale), ("residual", residual)):
+            if t is not None:
+                self._want(t, name, torch.float32)
+                if t.shape[-1] != width:
+                    raise KernelError(f"add_tanh_norm: {name} does not fit rows of {width}")
+        x_f32 = 0
+        if x is not None:
+            x_f32 = int(x.dtype == torch.float32 and dtype != torch.float32)
+            self._want(x, "x", torch.float32 if x_f32 else dtype)
+            if x.shape[1] != width or (residual is not None and x.shape != residual.shape):
+                raise KernelError("add_tanh_norm: the output does not fit the stream")
+        if rows is not None:
+            self._want(rows, "rows", torch.int32)
+            n_out, res_out = rows.shape[0], None
+        else:
+            n_out = src.shape[0]
+            res_out = residual if residual is not None else self.empty((n_out, width), torch.float32)
+        y = self.empty((n_out, width), dtype)
+        C, pos, weights, top = (experts.y, experts.pos, experts.weights, experts.top) if experts is not None else (None, None, None, 0)
+        fn = getattr(self.lib, "ptl_add_tanh_norm" + _suffix(dtype))
+        self._check(fn(_p(y), _p(res_out), _p(residual), _p(x), x_f32, _p(scale), _p(w), _p(b), float(alpha), _p(rows), n_out, width, _p(a1),
+                       _p(w0), _p(w1), count, float(eps), _p(C), _p(pos), _p(weights), top, self._stream()))
+        return y, res_out
+
+    def linear_add_tanh_norm(self, x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor, norm, scale: torch.Tensor) -> torch.Tensor:
+        """residual += scale * (x @ w^T), and the norm of the new residual."""
+        return self.add_tanh_norm(self.linear(x, w), residual, norm, scale=scale, dtype=x.dtype)[0]
+
+    def combine_experts_tanh_norm(self, rows: "ExpertRows", shared: Optional[torch.Tensor], residual: torch.Tensor, norm,
+                                  scale: torch.Tensor) -> torch.Tensor:
+        """residual += scale * (``shared`` + the weighted sum of the chosen experts' outputs), and the norm of the new residual."""
+        return self.add_tanh_norm(shared, residual, norm, scale=scale, dtype=rows.x.dtype, experts=rows)[0]
+
+    def linear_relu2(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """max(x @ w^T, 0)^2."""
+        y = self.linear(x, w)
+        self._check(getattr(self.lib, "ptl_relu2" + _suffix(y.dtype))(_p(y), y.numel(), self._stream()))
+        return y
+
+    def linear_each(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """[n, T, N]: x[i] @ w[i]^T for x [n, T, K] and w [n, N, K].  Many tokens in bfloat16: one batched product of the
+        library; otherwise the products one after another into their places."""
+        self._want(x, "x")
+        self._want(w, "w", x.dtype)
+        n, T, K = x.shape
+        N = w.shape[1]
+        if w.shape[0] != n or w.shape[2] != K:
+            raise KernelError("linear_each: shapes do not fit")
+        if x.dtype == torch.bfloat16 and T > 64 and self.library_products:
+            matmul = torch.backends.cuda.matmul
+            before = matmul.allow_bf16_reduced_precision_reduction
+            matmul.allow_bf16_reduced_precision_reduction = False
+            try:
+                return torch.bmm(x, w.transpose(1, 2))
+            finally:
+                matmul.allow_bf16_reduced_precision_reduction = before
+        plane = -(-T * N // 8) * 8                 # every result starts on a 16-byte boundary
+        out = self.empty((n, plane), x.dtype)[:, :T * N].unflatten(1, (T, N))
+        for i in range(n):
+            if x.dtype == torch.float32:
+                self._check(self.lib.ptl_gemm_simt_f32(_p(out[i]), _p(x[i]), _p(w[i]), T, N, K, K, K, N, 0, self._stream()))
+            elif self.gemm_tc(x[i], w[i], self.EPI_BF16, out=out[i]) is None:
+                out[i].copy_(self._library_mm(x[i], w[i], x.dtype))
+        return out
+
+    def token_shift(self, h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, ctx) -> torch.Tensor:
+        """[n, T, width]: h + (h' - h) * mu[i] for mu float32 [n, width], h' the row before of the same request; ``last`` float32
+        [slots, width] holds each request's last row and is moved on."""
+        self._want(h, "h")
+        self._want(mu, "mu", torch.float32)
+        self._want(last, "last rows", torch.float32)
+        T, width = h.shape
+        if mu.shape[1] != width or last.shape[1] != width:
+            raise KernelError("token_shift: shapes do not fit")
+        out = self.empty((mu.shape[0], T, width), h.dtype)
+        self._check(getattr(self.lib, "ptl_token_shift" + _suffix(h.dtype))(
+            _p(out), T * width, _p(h), _p(mu), mu.shape[0], T, width, _p(last), _p(ctx.q_start), _p(ctx.tok_req), _p(ctx.positions),
+            _p(ctx.state_slot), self._stream()))
+        return out
+
+    def wkv_scan(self, rkvg: torch.Tensor, z: torch.Tensor, w_bias: torch.Tensor, u: torch.Tensor, state: torch.Tensor, ctx, H: int,
+                 d: int) -> torch.Tensor:
+        """The recurrence of ``parts/wkv.py``: rkvg [>= 3, T, H*d] (r, k, v, ...); z float32 [T, H*d], the decay's argument before
+        its bias; u float32 [H*d]; state float32 [slots, H, d, d]; returns the heads' read-outs, float32 [T, H*d]."""
+        self._want(rkvg[0], "r")                  # (the planes may lie further apart than their size)
+        for name, t in (("z", z), ("w_bias", w_bias), ("u", u), ("state", state)):
+            self._want(t, name, torch.float32)
+        n, T = H * d, rkvg.shape[1]
+        if rkvg.shape[0] < 3 or rkvg.shape[2] != n or tuple(z.shape) != (T, n) or w_bias.numel() != n or u.numel() != n or \
+                tuple(state.shape[1:]) != (H, d, d):
+            raise KernelError("wkv_scan: shapes do not fit")
+        out = self.empty((T, n), torch.float32)
+        self._check(getattr(self.lib, "ptl_wkv_scan" + _suffix(rkvg.dtype))(
+            _p(out), _p(rkvg), rkvg.stride(0), _p(z), _p(w_bias), _p(u), _p(state), _p(ctx.q_start), _p(ctx.positions), _p(ctx.state_slot),
+            ctx.num_requests, H, d, self._stream()))
+        return out
+
+    def state_space_scan(self, xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, rate: torch.Tensor, D: torch.Tensor,
+                         state: torch.Tensor, ctx, H: int, G: int, n: int, dv: int) -> torch.Tensor:
+        """The recurrence of ``parts/state_space.py``: xbc [T, x: H*dv | B: G*n | C: G*n] after convolution; dt float32 [T, H] before
+        its bias; rate = exp(A_log) and D float32 [H]; state float32 [slots, H, n, dv]; returns y, float32 [T, H*dv]."""
+        self._want(xbc, "xbc")
+        for name, t in (("dt", dt), ("dt_bias", dt_bias), ("rate", rate), ("D", D), ("state", state)):
+            self._want(t, name, torch.float32)
+        T = xbc.shape[0]
+        if xbc.shape[1] != H * dv + 2 * G * n or tuple(dt.shape) != (T, H) or tuple(state.shape[1:]) != (H, n, dv) or \
+                any(t.numel() != H for t in (dt_bias, rate, D)):
+            raise KernelError("state_space_scan: shapes do not fit")
+        out = self.empty((T, H * dv), torch.float32)
+        self._check(getattr(self.lib, "ptl_state_space_scan" + _suffix(xbc.dtype))(
+            _p(out), _p(xbc), xbc.shape[1], _p(dt), _p(dt_bias), _p(rate), _p(D), _p(state), _p(ctx.q_start), _p(ctx.positions),
+            _p(ctx.state_slot), ctx.num_requests, H, G, n, dv, self._stream()))
+        return out
+
+    def gated_group_norm(self, y: torch.Tensor, gate: torch.Tensor, gate_column: int, weight: torch.Tensor, eps: float, groups: int,
+                         out: torch.Tensor, column: int, scale: float) -> None:
+        """With x = y * silu(gate[:, gate_column ..]): out[:, column ..] = x / rms(x's part) * weight * scale, a row being cut into
+        ``groups`` equal parts."""
+        self._want(y, "y", torch.float32)
+        self._want(weight, "norm weight", torch.float32)
+        self._want(gate, "gate")
+        self._want(out, "out", gate.dtype)
+        T, inner = y.shape
+        if weight.numel() != inner or inner % groups:
+            raise KernelError("gated_group_norm: shapes do not fit")
+        self._check(getattr(self.lib, "ptl_gated_group_norm" + _suffix(gate.dtype))(
+            _p(out), out.shape[1], int(column), _p(y), _p(weight), float(eps), _p(gate), gate.shape[1], int(gate_column), T, inner, int(groups),
+            float(scale), self._stream()))
+
+    def gated_lru(self, u: torch.Tensor, w_gates: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, yx: torch.Tensor,
+                  y_bias: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, column: int, scale: float) -> None:
+        """The recurrence of ``parts/gated_lru.py``: u [T, n]; w_gates [blocks, 2s, s] (a block's r rows, then its i rows);
+        gate_bias float32 [2, n]; rate float32 [n]; the gelu branch before its bias in the first n columns of yx; state float32
+        [slots, n]; the result times ``scale`` goes to columns ``column``.. of ``out``.  A 16-bit step of single tokens is one
+        kernel; otherwise the blocks' products come first (float32 results)."""
+        self._want(u, "u")
+        self._want(w_gates, "gate weights", u.dtype)
+        self._want(yx, "yx", u.dtype)
+        self._want(out, "out", u.dtype)
+        for name, t in (("gate bias", gate_bias), ("rate", rate), ("y bias", y_bias), ("state", state)):
+            self._want(t, name, torch.float32)
+        T, n = u.shape
+        B, two_s, s = w_gates.shape
+        if B * s != n or two_s != 2 * s or gate_bias.numel() != 2 * n or rate.numel() != n or y_bias.numel() != n or yx.shape[1] < n or \
+                tuple(state.shape[1:]) != (n,) or not 0 <= column <= out.shape[1] - n:
+            raise KernelError("gated_lru: shapes do not fit")
+        longest = int(getattr(ctx, "max_q_len", 0) or T)
+        if u.dtype == torch.bfloat16 and longest == 1:
+            rc = self.lib.ptl_gated_lru_single_bf16(_p(out), out.shape[1], int(column), _p(u), _p(w_gates), s, _p(gate_bias), _p(rate), _p(yx),
+                                                    yx.shape[1], _p(y_bias), _p(state), _p(ctx.tok_req), _p(ctx.positions),
+                                                    _p(ctx.state_slot), T, n, float(scale), self._stream())
+            if rc != -2:
+                self._check(rc)
+                return
+        if u.dtype == torch.bfloat16:
+            z = torch.bmm(u.view(T, B, s).transpose(0, 1), w_gates.transpose(1, 2), out_dtype=torch.float32)      # [B, T, 2s]
+            z_block, z_tok = T * 2 * s, 2 * s
+        else:
+            z = self.empty((T, B * 2 * s), torch.float32)
+            self.head_linear(u, s, 0, w_gates, z, 2 * s, 0, B)
+            z_block, z_tok = 2 * s, B * 2 * s
+        self._check(getattr(self.lib, "ptl_gated_lru_scan" + _suffix(u.dtype))(
+            _p(out), out.shape[1], int(column), _p(u), _p(z), z_block, z_tok, s, _p(gate_bias), _p(rate), _p(yx), yx.shape[1], _p(y_bias),
+            _p(state), _p(ctx.q_start), _p(ctx.positions), _p(ctx.state_slot), ctx.num_requests, longest, n, float(scale), self._stream()))
 
     def token_logprobs(self, logits: torch.Tensor, tokens: torch.Tensor) -> torch.Tensor:
         """log softmax(logits[row])[tokens[row]] as float32 [rows]."""
