@@ -6,6 +6,7 @@
     python bench.py --family sogalix      # the Sogalix decoder beside a Lilenex and a Llama of equal size
     python bench.py --family podizen      # the Podizen decoder beside a Lilenex and a Llama of equal size
     python bench.py --family nesisun      # the Nesisun decoder likewise
+    python bench.py --family gepilix      # the Gepilix decoder beside a Podizen and a Llama of equal size
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and context 4096, timed on
 the device with CUDA events around exactly K decode steps (a step = the engine's step function for
@@ -254,13 +255,35 @@ def _nesisun(width, layers, ff, vocab):
             "layers": [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": ff} if i % 2 == 0 else moe} for i in range(layers)]}
 
 
+def _gepilix(width, layers, ff, vocab):
+    """A Gepilix of sizes that resemble a real model's layers, three types in turn.  ``parallel``: attention in blocks of 512
+    positions (heads of 128, 4 query heads per kv head, one gate per head) beside a gated linear recurrence of ``width``
+    channels in blocks of 256; ``parallel_2``: attention with a window of 512 positions (same heads, half of every head
+    rotated, scaled frequencies) beside a state-space recurrence (inner = 2 width, heads of 64, 128 states, one group);
+    ``wkv``: heads of 64.  Feed-forwards alternate between the square of relu (two matrices, so 3/2 ff for the weights of a
+    gated one of ff) and 16 experts of ff/4, two per token, beside a shared one of ff/2."""
+    heads = width // 128
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "mask": {"size": 512}}
+    rot = {"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    mixers = {"parallel": {"left": att, "right": {"width": width, "blocks": width // 256, "conv": 4}},
+              "parallel_2": {"left": dict(att, rot=rot), "left_scale": 0.8, "right_scale": 0.6,
+                             "right": {"heads": width // 32, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}},
+              "wkv": {"heads": width // 64, "dim": 64}}
+    mlps = [{"kind": "dense", "ff": 3 * ff // 2},
+            {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 16, "top": 2}, "shared": {"ff": ff // 2}}]
+    kinds = ["parallel", "parallel_2", "wkv"]
+    return {"architecture": "Gepilix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": kinds[i % 3], "mixer": mixers[kinds[i % 3]], "mlp": mlps[i % 2]} for i in range(layers)]}
+
+
 FAMILIES = {"tibepel": (_tibepel, ["llama"]), "lilenex": (_lilenex, ["llama"]), "sogalix": (_sogalix, ["lilenex", "llama"]),
-            "podizen": (_podizen, ["lilenex", "llama"]), "nesisun": (_nesisun, ["lilenex", "llama"])}
+            "podizen": (_podizen, ["lilenex", "llama"]), "nesisun": (_nesisun, ["lilenex", "llama"]),
+            "gepilix": (_gepilix, ["podizen", "llama"])}
 
 
 def family_bench(args) -> int:
-    """``--family tibepel``, ``lilenex``, ``sogalix``, ``podizen`` or ``nesisun``: prefill (one step of 2,048 prompt tokens, as one prompt and as 8 prompts of 256) and decode
-    (8 requests at 1,024 tokens, a step with its sampling kernel) of that decoder and of a Llama decoder (for Sogalix, Podizen and Nesisun also a Lilenex decoder) of the
+    """``--family tibepel``, ``lilenex``, ``sogalix``, ``podizen``, ``nesisun`` or ``gepilix``: prefill (one step of 2,048 prompt tokens, as one prompt and as 8 prompts of 256) and decode
+    (8 requests at 1,024 tokens, a step with its sampling kernel) of that decoder and of a Llama decoder (for Sogalix, Podizen and Nesisun also a Lilenex decoder, for Gepilix a Podizen decoder) of the
     same width, depth, feed-forward size and vocabulary, on random weights, timed with CUDA events after warm-up; then one timed step of each kind with
     every operator bracketed by events, for the milliseconds by class of kernels.  One JSON line."""
     import torch

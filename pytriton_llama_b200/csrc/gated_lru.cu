@@ -3,11 +3,12 @@
 //   r = sigmoid(zr + b_r),  i = sigmoid(zi + b_i),  log a = -rate r   (rate = decay limit * softplus(lam) per channel)
 //   S <- a S + sqrt(1 - a^2) i u,      out = S * gelu_tanh(y + b_y) * scale
 //
-// 1 - a^2 is worked out as -expm1(2 log a), so that a channel that hardly decays keeps its input's weight.  All float32.
+// All float32.  The decay is kept as e = a - 1 = expm1(log a) and applied as S + (e S + ...): a channel that hardly decays would
+// lose the low bits of 1 - a, and with them a systematic share of its memory, if a were rounded.  1 - a^2 = -e (2 + e).
 //
 // gated_lru_scan, zr and zi given (products of many tokens, or float32): a block owns 32 neighbouring channels of one
 // request, its lanes; its NW warps take kLruTokens tokens each of a tile of NW * kLruTokens.  Every warp folds its tokens into
-// (product of a, result from zero), these meet in shared memory, every warp folds those before its own onto the state
+// (product of a, less one; result from zero), these meet in shared memory, every warp folds those before its own onto the state
 // and walks its tokens once more.  So a tile's loads are in flight together, and only the tiles follow one another.  The fold's
 // grouping depends on the place of a token within its portion, the arithmetic is a chain of fused multiply-adds either way.
 //
@@ -33,18 +34,19 @@ struct LruArgs {
 
 __device__ __forceinline__ float lru_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float lru_gelu(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
-// a and the share of u that enters the state
-__device__ __forceinline__ void lru_gates(float zr, float zi, float rate, float u, float& a, float& add) {
-  const float log_a = -rate * lru_sigmoid(zr);
-  a = expf(log_a);
-  add = sqrtf(-expm1f(2.0f * log_a)) * lru_sigmoid(zi) * u;
+// a - 1 and what enters the state
+__device__ __forceinline__ void lru_gates(float zr, float zi, float rate, float u, float& e, float& add) {
+  e = expm1f(-rate * lru_sigmoid(zr));
+  add = sqrtf(-e * (2.0f + e)) * lru_sigmoid(zi) * u;
 }
+// a S + add
+__device__ __forceinline__ float lru_step(float e, float S, float add) { return S + fmaf(e, S, add); }
 
 // Channel c of block b = c / s: its zr at z + b * z_block + t * z_tok + c % s, its zi s further on.
 template <typename T, int NW>
 __global__ void __launch_bounds__(NW * 32)
 gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long z_tok, int s, const LruArgs p) {
-  __shared__ float s_a[2][NW][32], s_b[2][NW][32];
+  __shared__ float s_e[2][NW][32], s_b[2][NW][32];
   pdl_wait();
   pdl_launch_dependents();
   const int r = blockIdx.y;
@@ -76,19 +78,19 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
   int buf = 0;
   for (int t0 = lo; t0 < hi; t0 += NW * kLruTokens, buf ^= 1) {
     const int first = t0 + warp * kLruTokens;
-    float a[kLruTokens], add[kLruTokens], g[kLruTokens];
-    float A = 1.f, B = 0.f;
+    float e[kLruTokens], add[kLruTokens], g[kLruTokens];
+    float E = 0.f, B = 0.f;
 #pragma unroll
     for (int k = 0; k < kLruTokens; ++k) {
-      lru_gates(zr[k] + br, zi[k] + bi, rate, to_f32(ru[k]), a[k], add[k]);
-      if (first + k >= hi) { a[k] = 1.f; add[k] = 0.f; }       // past the end: nothing changes
+      lru_gates(zr[k] + br, zi[k] + bi, rate, to_f32(ru[k]), e[k], add[k]);
+      if (first + k >= hi) { e[k] = 0.f; add[k] = 0.f; }       // past the end: nothing changes
       g[k] = lru_gelu(to_f32(ry[k]) + by) * p.scale;
-      A *= a[k];
-      B = fmaf(a[k], B, add[k]);
+      E = lru_step(e[k], E, e[k]);
+      B = lru_step(e[k], B, add[k]);
     }
     if (t0 + NW * kLruTokens < hi) fetch(t0 + NW * kLruTokens);        // in flight while the tile is folded and walked
     if constexpr (NW > 1) {
-      s_a[buf][warp][lane] = A;
+      s_e[buf][warp][lane] = E;
       s_b[buf][warp][lane] = B;
       __syncthreads();                                       // (the other buffer may still be read by warps behind)
     }
@@ -98,13 +100,13 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
 #pragma unroll
       for (int w = 0; w < NW; ++w) {
         if (w == warp) mine = all;
-        all = fmaf(s_a[buf][w][lane], all, s_b[buf][w][lane]);
+        all = lru_step(s_e[buf][w][lane], all, s_b[buf][w][lane]);
       }
       S = all;
     }
 #pragma unroll
     for (int k = 0; k < kLruTokens; ++k) {
-      mine = fmaf(a[k], mine, add[k]);
+      mine = lru_step(e[k], mine, add[k]);
       if (live && first + k < hi) out[(size_t)(first + k) * p.out_ld] = from_f32<T>(mine * g[k]);
     }
     if constexpr (NW == 1) S = mine;
@@ -161,10 +163,10 @@ gated_lru_single_kernel(const __nv_bfloat16* __restrict__ w, int s, const int* _
   if (lane >= tokens) return;
   const int r = tok_req[lane];
   if (r < 0 || p.state_slot[r] < 0) return;
-  float a, add;
-  lru_gates(zr + p.gate_bias[c], zi + p.gate_bias[p.n + c], p.rate[c], __bfloat162float(ub[(size_t)lane * p.n + e]), a, add);
+  float less, add;
+  lru_gates(zr + p.gate_bias[c], zi + p.gate_bias[p.n + c], p.rate[c], __bfloat162float(ub[(size_t)lane * p.n + e]), less, add);
   float* st = p.state + (size_t)p.state_slot[r] * p.n + c;
-  const float S = fmaf(a, p.positions[lane] == 0 ? 0.f : *st, add);
+  const float S = lru_step(less, p.positions[lane] == 0 ? 0.f : *st, add);
   *st = S;
   const float g = lru_gelu(__bfloat162float(((const __nv_bfloat16*)p.y)[(size_t)lane * p.y_ld + c]) + p.y_bias[c]) * p.scale;
   ((__nv_bfloat16*)p.out)[(size_t)lane * p.out_ld + p.column + c] = __float2bfloat16_rn(S * g);

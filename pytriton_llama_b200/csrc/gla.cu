@@ -49,6 +49,9 @@ struct GlaArgs {
 __device__ __forceinline__ float log_sigmoid_f32(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gla_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
+// exp(x), x <= 0, rounded once near 1: a decay of almost 1 acts a thousand times over, and any lean of its last bit with it
+__device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
+
 template <typename T, int RPL, int TB, int FORM>   // RPL rows per lane (d <= 8 * RPL), TB tokens per batch
 __global__ void __launch_bounds__(kGlaThreads)
 gla_scan_kernel(const GlaArgs p) {
@@ -130,7 +133,7 @@ gla_scan_kernel(const GlaArgs p) {
       if constexpr (FORM == kGlaStep) k *= s_step[buf][j];
       s_k[j][c_mine] = k;
       if constexpr (FORM == kGlaSigmoid) s_a[j][c_mine] = c_mine < d ? expf(log_sigmoid_f32(rz[i] + b_mine) * p.inv_tau) : 0.f;
-      if constexpr (FORM == kGlaBonus) s_a[j][c_mine] = c_mine < d ? expf(-expf(rz[i] + b_mine)) : 0.f;
+      if constexpr (FORM == kGlaBonus) s_a[j][c_mine] = c_mine < d ? decay_exp(-expf(rz[i] + b_mine)) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -145,7 +148,7 @@ gla_scan_kernel(const GlaArgs p) {
     if (FORM == kGlaStep && tid < TB) {    // (the walk over the batch before reads the other buffer)
       const float s = tid < nt ? gla_softplus(rdt + dt_bias) : 0.f;
       s_step[buf][tid] = s;
-      s_dec[buf][tid] = expf(-head_h * s);
+      s_dec[buf][tid] = decay_exp(-head_h * s);
     }
     __syncthreads();                       // the walk over the batch before is done with the staged tokens
     stage(buf);
