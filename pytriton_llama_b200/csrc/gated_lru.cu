@@ -6,10 +6,10 @@
 // All float32.  The decay is kept as e = a - 1 = expm1(log a) and applied as S + (e S + ...): a channel that hardly decays would
 // lose the low bits of 1 - a, and with them a systematic share of its memory, if a were rounded.  1 - a^2 = -e (2 + e).
 //
-// gated_lru_scan, zr and zi given (products of many tokens, or float32): a block owns 32 neighbouring channels of one
-// request, its lanes; its NW warps take kLruTokens tokens each of a tile of NW * kLruTokens.  Every warp folds its tokens into
-// (product of a, less one; result from zero), these meet in shared memory, every warp folds those before its own onto the state
-// and walks its tokens once more.  So a tile's loads are in flight together, and only the tiles follow one another.  The fold's
+// gated_lru_scan, zr and zi given (products of many tokens, or float32): a block owns kLruChannels neighbouring channels
+// of one request; its NG groups of as many threads take kLruTokens tokens each of a tile of NG * kLruTokens.  Every group folds its
+// tokens into (product of a, less one; result from zero), these meet in shared memory, every group folds those before its own onto
+// the state and walks its tokens once more.  So a tile's loads are in flight together, and only the tiles follow one another.  The fold's
 // grouping depends on the place of a token within its portion, the arithmetic is a chain of fused multiply-adds either way.
 //
 // gated_lru_single, one token per request, 16-bit: a warp per channel reads its two weight rows once and every token's block of
@@ -20,7 +20,8 @@
 
 namespace ptl {
 
-constexpr int kLruTokens = 8;       // tokens of a warp per tile
+constexpr int kLruTokens = 8;       // tokens of a group per tile
+constexpr int kLruChannels = 16;    // channels of a block (half a warp: a real model's few thousand channels then fill the SMs)
 
 struct LruArgs {
   void* out;                        // rows of out_ld elements, results at `column`
@@ -43,18 +44,18 @@ __device__ __forceinline__ void lru_gates(float zr, float zi, float rate, float 
 __device__ __forceinline__ float lru_step(float e, float S, float add) { return S + fmaf(e, S, add); }
 
 // Channel c of block b = c / s: its zr at z + b * z_block + t * z_tok + c % s, its zi s further on.
-template <typename T, int NW>
-__global__ void __launch_bounds__(NW * 32)
+template <typename T, int NG>
+__global__ void __launch_bounds__(NG * kLruChannels)
 gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long z_tok, int s, const LruArgs p) {
-  __shared__ float s_e[2][NW][32], s_b[2][NW][32];
+  __shared__ float s_e[2][NG][kLruChannels], s_b[2][NG][kLruChannels];
   pdl_wait();
   pdl_launch_dependents();
   const int r = blockIdx.y;
   const int lo = p.q_start[r], hi = p.q_start[r + 1];
   if (hi <= lo || p.state_slot[r] < 0) return;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const bool live = blockIdx.x * 32 + lane < p.n;
-  const int c = live ? blockIdx.x * 32 + lane : p.n - 1;       // lanes past the end shadow the last channel and store nothing
+  const int lane = threadIdx.x % kLruChannels, grp = threadIdx.x / kLruChannels;
+  const bool live = blockIdx.x * kLruChannels + lane < p.n;
+  const int c = live ? blockIdx.x * kLruChannels + lane : p.n - 1;       // lanes past the end shadow the last channel and store nothing
   const float* zc = z + (long long)(c / s) * z_block + c % s;
   const T* u = (const T*)p.u + c;
   const T* y = (const T*)p.y + c;
@@ -67,7 +68,7 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < kLruTokens; ++k) {
-      const int t = min(t0 + warp * kLruTokens + k, hi - 1);
+      const int t = min(t0 + grp * kLruTokens + k, hi - 1);
       zr[k] = zc[t * z_tok];
       zi[k] = zc[t * z_tok + s];
       ru[k] = u[(size_t)t * p.n];
@@ -76,8 +77,8 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
   };
   fetch(lo);
   int buf = 0;
-  for (int t0 = lo; t0 < hi; t0 += NW * kLruTokens, buf ^= 1) {
-    const int first = t0 + warp * kLruTokens;
+  for (int t0 = lo; t0 < hi; t0 += NG * kLruTokens, buf ^= 1) {
+    const int first = t0 + grp * kLruTokens;
     float e[kLruTokens], add[kLruTokens], g[kLruTokens];
     float E = 0.f, B = 0.f;
 #pragma unroll
@@ -88,30 +89,23 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
       E = lru_step(e[k], E, e[k]);
       B = lru_step(e[k], B, add[k]);
     }
-    if (t0 + NW * kLruTokens < hi) fetch(t0 + NW * kLruTokens);        // in flight while the tile is folded and walked
-    if constexpr (NW > 1) {
-      s_e[buf][warp][lane] = E;
-      s_b[buf][warp][lane] = B;
-      __syncthreads();                                       // (the other buffer may still be read by warps behind)
-    }
+    if (t0 + NG * kLruTokens < hi) fetch(t0 + NG * kLruTokens);        // in flight while the tile is folded and walked
+    s_e[buf][grp][lane] = E;
+    s_b[buf][grp][lane] = B;
+    __syncthreads();                                         // (the other buffer may still be read by groups behind)
     float mine = S;
-    if constexpr (NW > 1) {
-      float all = S;
 #pragma unroll
-      for (int w = 0; w < NW; ++w) {
-        if (w == warp) mine = all;
-        all = lru_step(s_e[buf][w][lane], all, s_b[buf][w][lane]);
-      }
-      S = all;
+    for (int w = 0; w < NG; ++w) {
+      if (w == grp) mine = S;
+      S = lru_step(s_e[buf][w][lane], S, s_b[buf][w][lane]);
     }
 #pragma unroll
     for (int k = 0; k < kLruTokens; ++k) {
       mine = lru_step(e[k], mine, add[k]);
       if (live && first + k < hi) out[(size_t)(first + k) * p.out_ld] = from_f32<T>(mine * g[k]);
     }
-    if constexpr (NW == 1) S = mine;
   }
-  if (live && warp == 0) *st = S;
+  if (live && grp == 0) *st = S;
 }
 
 constexpr int kLruSingleTokens = 32;   // tokens of a step that gated_lru_single takes at most (a lane each)
@@ -183,12 +177,12 @@ int gated_lru_scan(const float* z, long long z_block, long long z_tok, int s, co
   if (int rc = lru_check(p, s)) return rc;
   PTL_REQUIRE(requests >= 0 && requests <= 65535 && z_tok >= 2 * s && z_block >= 0, "gated_lru: bad sizes of the blocks' products");
   if (requests == 0) return 0;
-  const dim3 grid((p.n + 31) / 32, requests);
-#define PTL_LRU(NW) return launch_kernel("gated_lru_scan", gated_lru_scan_kernel<T, NW>, grid, dim3(NW * 32), 0, as_stream(stream), z, z_block, \
+  const dim3 grid((p.n + kLruChannels - 1) / kLruChannels, requests);
+#define PTL_LRU(NG) return launch_kernel("gated_lru_scan", gated_lru_scan_kernel<T, NG>, grid, dim3(NG * kLruChannels), 0, as_stream(stream), z, z_block, \
                                          z_tok, s, p)
-  if (longest <= kLruTokens) PTL_LRU(1);
-  if (longest <= 4 * kLruTokens) PTL_LRU(4);
-  PTL_LRU(16);
+  if (longest <= 2 * kLruTokens) PTL_LRU(2);
+  if (longest <= 8 * kLruTokens) PTL_LRU(8);
+  PTL_LRU(32);
 #undef PTL_LRU
 }
 

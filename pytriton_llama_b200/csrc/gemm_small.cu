@@ -13,7 +13,10 @@
 //     and go through the same epilogues as the tcgen05 product: bfloat16 or float32 store, or add
 //     into the float32 residual, optionally preparing the next RMS norm's input (xs = bfloat16(new
 //     residual * norm weight) and one sum of squares per token and block), and optionally finishing
-//     the norm before it (every output row scaled by rsqrt(mean of the token's squares + eps)).
+//     the norm before it (every output row scaled by rsqrt(mean of the token's squares + eps)); or the add is scaled by a
+//     vector and followed by the norm without statistics, y = tanh(alpha * residual) * w + b; or the square of relu is stored.
+// Several products of one shape (their operands and results `*_plane` elements apart) can go in one launch, blockIdx.y
+// being the product.
 // Sizes: M <= 8, K % 8 == 0, and as many blocks as are resident at once (the launcher says no
 // otherwise and the caller takes the tcgen05 product).
 #include "mma_utils.cuh"
@@ -40,6 +43,12 @@ struct SmallGemmParams {
   const float* scale_sumsq;
   int scale_slots, scale_ld;
   float scale_eps, scale_inv_n;
+  // add epilogue: a scale per feature, then y = tanh(alpha * residual) * w + b (all null otherwise)
+  const float *tail_scale, *tail_w, *tail_b;
+  float tail_alpha;
+  __nv_bfloat16* tail_y;
+  int relu2;                         // epilogue 0: the square of max(result, 0)
+  long long x_plane, w_plane, out_plane;
   unsigned long long* timeline;
   int timeline_kind;
 };
@@ -47,7 +56,13 @@ struct SmallGemmParams {
 // EPI: 0 bfloat16 store, 1 float32 store, 2 add into the float32 residual
 template <int EPI>
 __global__ void __launch_bounds__(kSmallWarps * 32, 3)
-gemm_small_kernel(const SmallGemmParams p) {
+gemm_small_kernel(const SmallGemmParams p_in) {
+  SmallGemmParams p = p_in;
+  if (EPI == 0) {
+    p.X += (long long)blockIdx.y * p.x_plane;
+    p.W += (long long)blockIdx.y * p.w_plane;
+    p.out = (__nv_bfloat16*)p.out + (long long)blockIdx.y * p.out_plane;
+  }
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0 && p.timeline) { timeline_stamp(p.timeline, 0); if (blockIdx.x == 0) p.timeline[0] = p.timeline_kind; }
@@ -84,8 +99,9 @@ gemm_small_kernel(const SmallGemmParams p) {
   const int e_tok = tid / kSmallRows, e_row = tid % kSmallRows;
   const int n = n0 + e_row;
   const bool e_valid = tid < kSmallRows * kSmallTokens && e_tok < p.M && n < p.N;
-  float have = 0.f, nw = 0.f;
+  float have = 0.f, nw = 0.f, t_scale = 1.f, t_w = 0.f, t_b = 0.f;
   if (EPI == 2 && e_valid) {
+    if (p.tail_y) { t_scale = __ldg(p.tail_scale + n); t_w = __ldg(p.tail_w + n); t_b = __ldg(p.tail_b + n); }
     have = __ldcg((const float*)p.out + (size_t)e_tok * p.ld_out + n);
     if (p.xs) nw = __ldg(p.norm_w + n);
   }
@@ -134,12 +150,16 @@ gemm_small_kernel(const SmallGemmParams p) {
     for (int w = 0; w < kSmallWarps; ++w) v += s_part[(w * kSmallRows + e_row) * kSmallTokens + e_tok];
     if (p.scale_sumsq) v *= s_scale[e_tok];
     if (e_valid) {
-      if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)e_tok * p.ld_out + n] = __float2bfloat16_rn(v);
+      if (EPI == 0) {
+        if (p.relu2) { v = fmaxf(v, 0.f); v *= v; }
+        ((__nv_bfloat16*)p.out)[(size_t)e_tok * p.ld_out + n] = __float2bfloat16_rn(v);
+      }
       else if (EPI == 1) ((float*)p.out)[(size_t)e_tok * p.ld_out + n] = v;
       else {
-        r_new = have + v;
+        r_new = fmaf(t_scale, v, have);
         ((float*)p.out)[(size_t)e_tok * p.ld_out + n] = r_new;
         if (p.xs) p.xs[(size_t)e_tok * p.xs_ld + n] = __float2bfloat16_rn(r_new * nw);
+        if (p.tail_y) p.tail_y[(size_t)e_tok * p.N + n] = __float2bfloat16_rn(fmaf(tanhf(p.tail_alpha * r_new), t_w, t_b));
       }
     }
     if (EPI == 2 && p.xs) {
@@ -155,10 +175,10 @@ gemm_small_kernel(const SmallGemmParams p) {
 }
 
 template <int EPI>
-static int launch_small(const SmallGemmParams& p, int blocks, size_t smem, cudaStream_t stream) {
+static int launch_small(const SmallGemmParams& p, int blocks, size_t smem, cudaStream_t stream, int products = 1) {
   static SmemRaised raised = {};
   if (int rc = raise_shared_memory("gemm_small", gemm_small_kernel<EPI>, 100 * 1024, raised)) return rc;
-  return launch_kernel("gemm_small", gemm_small_kernel<EPI>, dim3(blocks), dim3(kSmallWarps * 32), smem, stream, p);
+  return launch_kernel("gemm_small", gemm_small_kernel<EPI>, dim3(blocks, products), dim3(kSmallWarps * 32), smem, stream, p);
 }
 
 }  // namespace ptl
@@ -167,10 +187,12 @@ static int launch_small(const SmallGemmParams& p, int blocks, size_t smem, cudaS
 // multiple of 8, rows too long for three blocks per SM, or more blocks than are resident at once):
 // the caller then takes the tcgen05 product.  Arguments as ptl_gemm_tc_bf16_norm (epi 0, 1 or 2);
 // with `xs` a token gets one slot of `sumsq` per 8 features, *slots_out = ceil(N / 8).
-PTL_EXPORT int ptl_gemm_small_bf16(void* out, const void* X, const void* W, int M, int N, int K, int ld_out, int epi,
-                                   void* xs, const float* norm_w, float* sumsq, int sumsq_ld, int* slots_out,
-                                   const float* scale_sumsq, int scale_slots, int scale_ld, float scale_eps, void* stream) {
+static int gemm_small_impl(void* out, const void* X, const void* W, int M, int N, int K, int ld_out, int epi, void* xs,
+                           const float* norm_w, float* sumsq, int sumsq_ld, int* slots_out, const float* scale_sumsq, int scale_slots,
+                           int scale_ld, float scale_eps, void* stream, const ptl::SmallGemmParams* more = nullptr, int products = 1) {
   using namespace ptl;
+  const int relu2 = epi == 6;
+  if (relu2) epi = 0;
   PTL_REQUIRE(M >= 0 && N > 0 && K > 0 && ld_out > 0, "gemm_small: bad sizes M=%d N=%d K=%d", M, N, K);
   if (M > kSmallTokens || K % 8 != 0 || epi < 0 || epi > 2) return -2;
   if (M == 0) return 0;
@@ -178,6 +200,11 @@ PTL_EXPORT int ptl_gemm_small_bf16(void* out, const void* X, const void* W, int 
   SmallGemmParams p{};
   p.out = out; p.X = (const __nv_bfloat16*)X; p.W = (const __nv_bfloat16*)W;
   p.M = M; p.N = N; p.K = K; p.ld_out = ld_out;
+  p.relu2 = relu2;
+  if (more) {
+    p.tail_scale = more->tail_scale; p.tail_w = more->tail_w; p.tail_b = more->tail_b; p.tail_alpha = more->tail_alpha; p.tail_y = more->tail_y;
+    p.x_plane = more->x_plane; p.w_plane = more->w_plane; p.out_plane = more->out_plane;
+  }
   p.k_per_warp = ((K + kSmallWarps - 1) / kSmallWarps + 15) / 16 * 16;
   const int row_elems = kSmallWarps * p.k_per_warp + kSmallPad;
   const size_t smem = (size_t)(kSmallRows + kSmallTokens) * row_elems * 2 + (kSmallWarps * kSmallRows * kSmallTokens + kSmallTokens) * 4;
@@ -206,8 +233,36 @@ PTL_EXPORT int ptl_gemm_small_bf16(void* out, const void* X, const void* W, int 
   p.timeline_kind = 20 + epi;
   cudaStream_t s = as_stream(stream);
   switch (epi) {
-    case 0: return launch_small<0>(p, blocks, smem, s);
+    case 0: return launch_small<0>(p, blocks, smem, s, products);
     case 1: return launch_small<1>(p, blocks, smem, s);
     default: return launch_small<2>(p, blocks, smem, s);
   }
+}
+
+PTL_EXPORT int ptl_gemm_small_bf16(void* out, const void* X, const void* W, int M, int N, int K, int ld_out, int epi,
+                                   void* xs, const float* norm_w, float* sumsq, int sumsq_ld, int* slots_out,
+                                   const float* scale_sumsq, int scale_slots, int scale_ld, float scale_eps, void* stream) {
+  return gemm_small_impl(out, X, W, M, N, K, ld_out, epi, xs, norm_w, sumsq, sumsq_ld, slots_out, scale_sumsq, scale_slots, scale_ld,
+                         scale_eps, stream);
+}
+
+// residual [M, N] (float32, in place) += scale * (X W^T) and y = bfloat16(tanh(alpha * residual) * w + b) [M, N].
+PTL_EXPORT int ptl_gemm_small_tanh_norm_bf16(float* residual, const void* X, const void* W, int M, int N, int K, const float* scale,
+                                             const float* w, const float* b, float alpha, void* y, void* stream) {
+  using namespace ptl;
+  PTL_REQUIRE(scale && w && b && y, "gemm_small: the scaled add with its norm needs scale, weight, bias and a result");
+  SmallGemmParams more{};
+  more.tail_scale = scale; more.tail_w = w; more.tail_b = b; more.tail_alpha = alpha; more.tail_y = (__nv_bfloat16*)y;
+  return gemm_small_impl(residual, X, W, M, N, K, N, 2, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0.f, stream, &more);
+}
+
+// `products` products of one shape: out + i out_plane = (X + i x_plane) (W + i w_plane)^T, bfloat16 [M, N].
+PTL_EXPORT int ptl_gemm_small_each_bf16(void* out, long long out_plane, const void* X, long long x_plane, const void* W, long long w_plane,
+                                        int products, int M, int N, int K, void* stream) {
+  using namespace ptl;
+  PTL_REQUIRE(products >= 1 && products <= 65535, "gemm_small: %d products", products);
+  if (x_plane % 8 != 0 || w_plane % 8 != 0) return -2;
+  SmallGemmParams more{};
+  more.x_plane = x_plane; more.w_plane = w_plane; more.out_plane = out_plane;
+  return gemm_small_impl(out, X, W, M, N, K, N, 0, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0.f, stream, &more, products);
 }

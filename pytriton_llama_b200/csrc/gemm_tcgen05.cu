@@ -66,7 +66,7 @@ PTL_EXPORT int ptl_gemm_tc_k_parts(int M, int N, int K) {
 }
 
 // out: epi 0 bf16 [M,N]; 1 float32 [M,N]; 2 float32 [M,N] added to in place; 3 bf16 [M,N/2], silu(gate) * up of weight
-// rows that alternate gate, up; 5 the same with the tanh form of gelu.
+// rows that alternate gate, up; 5 the same with the tanh form of gelu; 6 bf16 [M,N], the square of max(result, 0).
 // Returns -2 when the sizes are not ones this kernel takes (K % 8 != 0 or K < 64), so that the caller
 // can use another product.  `splits_hint` > 0 forces the number of K splits when M <= 64 (1, 2, 4 or 8);
 // when M > 64 it asks for that many parts of the K range, whose partial sums are stored one after
@@ -83,7 +83,8 @@ static int gemm_tc_impl(void* out, const void* X, const void* W, int M, int N, i
                         int* status, int splits_hint, void* xs, const float* norm_w, float* sumsq,
                         int sumsq_ld, int* slots_out, const float* scale_sumsq, int scale_slots,
                         int scale_ld, float scale_eps, const ptl::GemmParams* rope, void* stream,
-                        unsigned poll_limit = ptl::kPollLimit, int withhold_first_load = 0) {
+                        unsigned poll_limit = ptl::kPollLimit, int withhold_first_load = 0,
+                        const ptl::GemmParams* tail = nullptr) {
   using namespace ptl;
   PTL_REQUIRE(M >= 0 && N > 0 && K > 0 && ld_out > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
   if (K % 8 != 0 || K < kTileK) return -2;
@@ -94,6 +95,14 @@ static int gemm_tc_impl(void* out, const void* X, const void* W, int M, int N, i
     epi = 3;
     p.gate_a = 1.5957691216057308f;      // 2 sqrt(2 / pi)
     p.gate_b = 0.044715f * p.gate_a;
+  }
+  if (epi == 6) {
+    epi = 0;
+    p.relu2 = 1;
+  }
+  if (tail) {
+    if (epi != 2 || M > 64) return -2;
+    p.tail_scale = tail->tail_scale; p.tail_w = tail->tail_w; p.tail_b = tail->tail_b; p.tail_alpha = tail->tail_alpha; p.tail_y = tail->tail_y;
   }
   PTL_REQUIRE(epi != 3 || N % 2 == 0, "gemm_tc: the gate*up epilogue needs an even number of weight rows");
   if (M == 0) return 0;
@@ -186,7 +195,7 @@ PTL_EXPORT int ptl_gemm_tc_bf16_norm(void* out, const void* X, const void* W, in
                                      int* status, int splits_hint, void* xs, const float* norm_w, float* sumsq,
                                      int sumsq_ld, int* slots_out, const float* scale_sumsq, int scale_slots,
                                      int scale_ld, float scale_eps, void* stream) {
-  PTL_REQUIRE((epi >= 0 && epi <= 3) || epi == 5, "gemm_tc: unknown epilogue %d", epi);
+  PTL_REQUIRE((epi >= 0 && epi <= 3) || epi == 5 || epi == 6, "gemm_tc: unknown epilogue %d", epi);
   return gemm_tc_impl(out, X, W, M, N, K, ld_out, epi, status, splits_hint, xs, norm_w, sumsq, sumsq_ld, slots_out, scale_sumsq,
                       scale_slots, scale_ld, scale_eps, nullptr, stream);
 }
@@ -207,6 +216,18 @@ PTL_EXPORT int ptl_gemm_tc_bf16_qkv_rope(void* out, const void* X, const void* W
   rope.rope_table = (const float2*)table; rope.rope_slots = slots; rope.rope_cache = (__nv_bfloat16*)cache;
   rope.rope_nq = nq; rope.rope_nkv = nkv; rope.rope_d = d; rope.rope_page = page_size; rope.rope_num_slots = num_slots;
   return gemm_tc_impl(out, X, W, M, N, K, N, 4, status, 0, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0.f, &rope, stream);
+}
+
+// A step of at most 64 tokens: residual [M, N] (float32, in place) += scale * (X W^T) and y = bfloat16(tanh(alpha * residual) * w
+// + b) [M, N].  -2 where the sizes are not taken.
+PTL_EXPORT int ptl_gemm_tc_tanh_norm_bf16(float* residual, const void* X, const void* W, int M, int N, int K, int* status,
+                                          const float* scale, const float* w, const float* b, float alpha, void* y, void* stream) {
+  using namespace ptl;
+  PTL_REQUIRE(scale && w && b && y, "gemm_tc: the scaled add with its norm needs scale, weight, bias and a result");
+  GemmParams tail{};
+  tail.tail_scale = scale; tail.tail_w = w; tail.tail_b = b; tail.tail_alpha = alpha; tail.tail_y = (__nv_bfloat16*)y;
+  return gemm_tc_impl(residual, X, W, M, N, K, N, 2, status, 0, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0.f, nullptr, stream,
+                      kPollLimit, 0, &tail);
 }
 
 PTL_EXPORT int ptl_gemm_tc_bf16(void* out, const void* X, const void* W, int M, int N, int K, int ld_out, int epi,

@@ -15,6 +15,7 @@
 //     rank order and runs the epilogue on them.
 //
 // Epilogues: 0 store bfloat16, 1 store float32, 2 add into a float32 residual [M,N] in place,
+// (with few tokens optionally times a vector, and with the norm that follows where that is tanh(alpha x) w + b),
 // 3 SiLU(gate)*up where the rows of W alternate gate_j, up_j (out is [M, N/2] bfloat16).
 //
 // Warp roles (320 threads): warp 0 TMA producer, warp 1 TMEM allocation + MMA issue (with few tokens
@@ -80,6 +81,12 @@ struct GemmParams {
   // run out, and the test sees the status word, the drained roles and the block's clean exit.
   uint32_t poll_limit;
   int withhold_first_load;
+  // Few tokens, add epilogue: residual += tail_scale * result instead of the plain sum, and the norm without statistics that
+  // reads it next, tail_y = bfloat16(tanh(tail_alpha * residual) * tail_w + tail_b) [tokens, rows] (all null otherwise).
+  const float *tail_scale, *tail_w, *tail_b;
+  float tail_alpha;
+  __nv_bfloat16* tail_y;
+  int relu2;                      // epilogue 0: the square of max(result, 0) is stored
   float gate_a, gate_b;           // epilogue 3: the gate's activation (gate_act)
   unsigned long long* timeline;   // measurements: where the first and the last block stamp %globaltimer (null: nowhere)
   int timeline_kind;
@@ -132,6 +139,17 @@ __device__ __forceinline__ float gate_act(const GemmParams& p, float g) {
   return __fdividef(g, 1.0f + __expf(-g * fmaf(p.gate_b, g * g, p.gate_a)));
 }
 
+__device__ __forceinline__ float plain_act(const GemmParams& p, float v) {
+  if (!p.relu2) return v;
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
+// What the add epilogue adds for feature n, and what it does with the new residual r of (token, n).
+__device__ __forceinline__ float tail_term(const GemmParams& p, int n, float v) { return p.tail_y ? v * __ldg(p.tail_scale + n) : v; }
+__device__ __forceinline__ void tail_store(const GemmParams& p, int n, int tok, float r) {
+  if (p.tail_y) p.tail_y[(size_t)tok * p.rows + n] = __float2bfloat16_rn(fmaf(tanhf(p.tail_alpha * r), __ldg(p.tail_w + n), __ldg(p.tail_b + n)));
+}
+
 // ---------------------------------------------------------------- epilogue of one row's 16 accumulators
 // Normal mode: `row` is a token, columns c0..c0+15 are features.
 template <int EPI>
@@ -166,7 +184,7 @@ __device__ __forceinline__ void store_normal(const GemmParams& p, int row, int c
         uint32_t* w = reinterpret_cast<uint32_t*>(&pk);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          __nv_bfloat162 t = __floats2bfloat162_rn(v[8 * h + 2 * j], v[8 * h + 2 * j + 1]);
+          __nv_bfloat162 t = __floats2bfloat162_rn(plain_act(p, v[8 * h + 2 * j]), plain_act(p, v[8 * h + 2 * j + 1]));
           w[j] = *reinterpret_cast<uint32_t*>(&t);
         }
         *reinterpret_cast<uint4*>(o + 8 * h) = pk;
@@ -174,7 +192,7 @@ __device__ __forceinline__ void store_normal(const GemmParams& p, int row, int c
     } else {
 #pragma unroll
       for (int j = 0; j < 16; ++j)
-        if (c0 + j < n_total) o[j] = __float2bfloat16_rn(v[j]);
+        if (c0 + j < n_total) o[j] = __float2bfloat16_rn(plain_act(p, v[j]));
     }
   } else {   // EPI 1 (store float32) or 2 (add into float32)
     float* o = (float*)p.out + out_row * p.ld_out + c0;
@@ -214,8 +232,9 @@ __device__ __forceinline__ void add_and_emit(const GemmParams& p, int n, int tok
   float r = 0.f;
   if (valid) {
     float* o = (float*)p.out + (size_t)tok * p.ld_out + n;
-    r = (fetched ? have : __ldcg(o)) + v;
+    r = (fetched ? have : __ldcg(o)) + tail_term(p, n, v);
     *o = r;
+    tail_store(p, n, tok, r);
     if (p.xs) p.xs[(size_t)tok * p.xs_ld + n] = __float2bfloat16_rn(r * (fetched ? norm_w : __ldg(p.norm_w + n)));
   }
   if (p.xs) {
@@ -239,7 +258,7 @@ __device__ __forceinline__ void store_swapped(const GemmParams& p, int row, int 
     } else if (EPI == 2) {
       add_and_emit(p, n, tok, v[j], false, 0.f, threadIdx.x & 31);
     } else if (n_ok && tok < p.cols) {
-      if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n] = __float2bfloat16_rn(v[j]);
+      if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n] = __float2bfloat16_rn(plain_act(p, v[j]));
       else ((float*)p.out)[(size_t)tok * p.ld_out + n] = v[j];
     }
   }
@@ -249,7 +268,7 @@ __device__ __forceinline__ void store_swapped(const GemmParams& p, int row, int 
 template <int EPI>
 __device__ __forceinline__ void store_swapped_one(const GemmParams& p, int n, int tok, float v, float up) {
   if (n >= p.rows || tok >= p.cols) return;
-  if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n] = __float2bfloat16_rn(v);
+  if (EPI == 0) ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n] = __float2bfloat16_rn(plain_act(p, v));
   else if (EPI == 1) ((float*)p.out)[(size_t)tok * p.ld_out + n] = v;
   else if (EPI == 2) ((float*)p.out)[(size_t)tok * p.ld_out + n] += v;
   else ((__nv_bfloat16*)p.out)[(size_t)tok * p.ld_out + n / 2] = __float2bfloat16_rn(gate_act(p, v) * up);
@@ -767,6 +786,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_row, const __grid_constan
           if (EPI == 2) {
             // residual += v; with p.xs the next norm's input and the sum of squares of 16 features (four lanes) go out too
             float rn[4] = {0.f, 0.f, 0.f, 0.f};
+            if (p.tail_y) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) if (n + j < p.rows && col < p.cols) v[j] = tail_term(p, n + j, v[j]);
+            }
             if (live && vec_out) {
               float4* o = reinterpret_cast<float4*>((float*)p.out + (size_t)col * p.ld_out + n);
               const float4 have = i == 0 ? res0 : __ldcg(o);
@@ -790,6 +813,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_row, const __grid_constan
                 }
               }
             }
+            if (p.tail_y) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) if (n + j < p.rows && col < p.cols) tail_store(p, n + j, col, rn[j]);
+            }
             if (p.xs) {
               float sq = (rn[0] * rn[0] + rn[1] * rn[1]) + (rn[2] * rn[2] + rn[3] * rn[3]);
               sq += __shfl_xor_sync(0xffffffffu, sq, 1);       // the four lanes that hold 16 neighbouring features of this token
@@ -812,12 +839,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_row, const __grid_constan
               __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)col * p.ld_out + n;
               if (live && vec_out) {
                 uint2 pk;
-                pk.x = pack_bf16x2(v[0], v[1]);
-                pk.y = pack_bf16x2(v[2], v[3]);
+                pk.x = pack_bf16x2(plain_act(p, v[0]), plain_act(p, v[1]));
+                pk.y = pack_bf16x2(plain_act(p, v[2]), plain_act(p, v[3]));
                 *reinterpret_cast<uint2*>(o) = pk;
               } else {
 #pragma unroll
-                for (int j = 0; j < 4; ++j) if (n + j < p.rows) o[j] = __float2bfloat16_rn(v[j]);
+                for (int j = 0; j < 4; ++j) if (n + j < p.rows) o[j] = __float2bfloat16_rn(plain_act(p, v[j]));
               }
             } else {
               float* o = (float*)p.out + (size_t)col * p.ld_out + n;

@@ -84,6 +84,91 @@ __global__ void causal_conv_kernel(T* __restrict__ out, const T* __restrict__ x,
   out[(size_t)t * channels + c] = from_f32<T>(silu ? silu_f32(acc) : acc);
 }
 
+// The same for steps with portions, TAPS taps and rows of whole pairs: a thread takes two neighbouring channels of kConvTokens
+// tokens and keeps the last inputs in registers; eight rows are requested together.
+constexpr int kConvTokens = 32;
+template <typename T> struct ConvPair;
+template <> struct ConvPair<float> {
+  float2 raw;
+  __device__ __forceinline__ float2 get() const { return raw; }
+};
+template <> struct ConvPair<__nv_bfloat16> {
+  __nv_bfloat162 raw;
+  __device__ __forceinline__ float2 get() const { return __bfloat1622float2(raw); }
+};
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+causal_conv_rows_kernel(T* __restrict__ out, const T* __restrict__ x, int ld, int column, int channels, const float* __restrict__ w,
+                        const float* __restrict__ b, const float* __restrict__ state, const int* __restrict__ q_start,
+                        const int* __restrict__ tok_req, const int* __restrict__ positions, const int* __restrict__ state_slot,
+                        int silu, const float* __restrict__ in_bias, int tokens) {
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 2;
+  const int first = blockIdx.x * kConvTokens, end = min(first + kConvTokens, tokens);
+  float2 wt[TAPS], own = make_float2(0.f, 0.f), bias = make_float2(0.f, 0.f);
+  if (c < channels) {        // a model's weights depend on no earlier kernel
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) wt[k] = make_float2(w[(size_t)c * TAPS + k], w[(size_t)(c + 1) * TAPS + k]);
+    if (in_bias) own = make_float2(in_bias[c], in_bias[c + 1]);
+    if (b) bias = make_float2(b[c], b[c + 1]);
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  if (c >= channels) return;
+  const T* xc = x + column + c;
+  auto row = [&](int t) {
+    ConvPair<T> v;
+    v.raw = *reinterpret_cast<const decltype(v.raw)*>(xc + (size_t)t * ld);
+    return v;
+  };
+  float2 past[TAPS > 1 ? TAPS - 1 : 1];      // the inputs before the token, oldest first
+  int req = -1;                              // whose inputs they are
+  for (int t0 = first; t0 < end; t0 += 8) {
+    ConvPair<T> raw[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) raw[k] = row(min(t0 + k, end - 1));
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int t = t0 + k;
+      if (t >= end) break;
+      const int r = tok_req[t];
+      if (r < 0) { req = -1; continue; }
+      if (r != req) {                        // the thread's first token, or a request's: fetch what lies before it
+        req = r;
+        const int in_step = t - q_start[r], pos = positions[t];
+        const float* st = state + (size_t)state_slot[r] * (TAPS > 1 ? TAPS - 1 : 1) * channels + c;
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int back = TAPS - 1 - j;
+          past[j] = make_float2(0.f, 0.f);
+          if (back <= in_step) {
+            past[j] = row(t - back).get();
+            past[j].x += own.x; past[j].y += own.y;
+          } else if (back <= pos) {
+            const float* s = st + (size_t)(j + in_step) * channels;
+            past[j] = make_float2(s[0], s[1]);
+          }
+        }
+      }
+      float2 now = raw[k].get();
+      now.x += own.x; now.y += own.y;
+      float2 acc = bias;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        acc.x = fmaf(wt[j].x, past[j].x, acc.x);
+        acc.y = fmaf(wt[j].y, past[j].y, acc.y);
+        past[j] = j + 1 < TAPS - 1 ? past[j + 1] : now;
+      }
+      acc.x = fmaf(wt[TAPS - 1].x, now.x, acc.x);
+      acc.y = fmaf(wt[TAPS - 1].y, now.y, acc.y);
+      if (silu) { acc.x = silu_f32(acc.x); acc.y = silu_f32(acc.y); }
+      T* dst = out + (size_t)t * channels + c;
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = acc;
+      else *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(acc.x, acc.y);
+    }
+  }
+}
+
 // The state after the step: the last taps - 1 inputs of each request.  New entry j takes the step's row
 // n - (taps - 1) + j, or, where that lies before the step, the old entry j + n (zero before position 0).
 // Ascending j reads only entries that have not been rewritten yet.
@@ -515,7 +600,17 @@ int causal_conv(void* out, const void* x, int ld, int column, int channels, cons
   PTL_REQUIRE(tiles.x <= 65535, "causal_conv: too many channels (%d)", channels);
   // a step of single tokens (as many rows as requests, each request's rows being one): one kernel reads and moves the state
   float* state_out = (single_tokens && taps > 1) ? state : nullptr;
-  if (int rc = launch_kernel("causal_conv", causal_conv_kernel<T>, dim3(tokens, tiles.x), block, 0, as_stream(stream), (T*)out,
+  const bool pairs = channels % 2 == 0 && ld % 2 == 0 && column % 2 == 0 && aligned16(x) && aligned16(out);
+  if (!state_out && pairs && taps >= 2 && taps <= 4) {
+    const dim3 grid((tokens + kConvTokens - 1) / kConvTokens, (channels + 255) / 256);
+#define PTL_CONV_ROWS(TAPS)                                                                                                     \
+    if (int rc = launch_kernel("causal_conv_rows", causal_conv_rows_kernel<T, TAPS>, grid, block, 0, as_stream(stream), (T*)out, \
+                               (const T*)x, ld, column, channels, w, b, (const float*)state, q_start, tok_req, positions,       \
+                               state_slot, silu, in_bias, tokens))                                                              \
+      return rc;
+    if (taps == 2) { PTL_CONV_ROWS(2) } else if (taps == 3) { PTL_CONV_ROWS(3) } else { PTL_CONV_ROWS(4) }
+#undef PTL_CONV_ROWS
+  } else if (int rc = launch_kernel("causal_conv", causal_conv_kernel<T>, dim3(tokens, tiles.x), block, 0, as_stream(stream), (T*)out,
                              (const T*)x, ld, column, channels, w, b, taps, (const float*)state, q_start, tok_req, positions,
                              state_slot, silu, state_out, in_bias))
     return rc;

@@ -209,6 +209,12 @@ def load_library() -> ctypes.CDLL:
     lib.ptl_lowrank_tanh_linear.restype = _c_int
     lib.ptl_head_linear_few_bf16.argtypes = _SIGNATURES["ptl_head_linear"]
     lib.ptl_head_linear_few_bf16.restype = _c_int
+    lib.ptl_gemm_small_tanh_norm_bf16.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _c_f, _ptr, _ptr]
+    lib.ptl_gemm_small_tanh_norm_bf16.restype = _c_int
+    lib.ptl_gemm_small_each_bf16.argtypes = [_ptr, _c_ll, _ptr, _c_ll, _ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _ptr]
+    lib.ptl_gemm_small_each_bf16.restype = _c_int
+    lib.ptl_gemm_tc_tanh_norm_bf16.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr, _ptr, _ptr, _ptr, _c_f, _ptr, _ptr]
+    lib.ptl_gemm_tc_tanh_norm_bf16.restype = _c_int
     lib.ptl_gated_lru_single_bf16.argtypes = [_ptr, _c_int, _c_int, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr,
                                               _ptr, _c_int, _c_int, _c_f, _ptr]
     lib.ptl_gated_lru_single_bf16.restype = _c_int
@@ -562,7 +568,7 @@ class CudaOps:
         return y
 
     # epilogues of the tensor-core product
-    EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SILU_MUL, EPI_GELU_MUL = 0, 1, 2, 3, 5
+    EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SILU_MUL, EPI_GELU_MUL, EPI_RELU2 = 0, 1, 2, 3, 5, 6
     GATE_EPILOGUES = {"silu": EPI_SILU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
     def _tc_status_word(self):
@@ -573,7 +579,7 @@ class CudaOps:
     def gemm_tc(self, x, w: torch.Tensor, epi: int = 0, out: Optional[torch.Tensor] = None,
                 splits: int = 0, emit_norm=None, column: int = 0):
         """x[M,K] @ w[N,K]^T in bfloat16 on the tcgen05 tensor cores with a fused epilogue.
-        ``epi``: EPI_BF16 -> [M,N] bfloat16; EPI_F32 -> [M,N] float32; EPI_ADD_F32 adds into ``out``
+        ``epi``: EPI_BF16 -> [M,N] bfloat16 (EPI_RELU2: the square of max(result, 0)); EPI_F32 -> [M,N] float32; EPI_ADD_F32 adds into ``out``
         (float32 [M,N], in place); EPI_SILU_MUL, EPI_GELU_MUL -> [M,N/2] bfloat16 for weights whose rows alternate
         gate_j, up_j (written to columns ``column``.. of ``out`` where that is given).  ``x`` may be a ``NormedActivation``: its row scale is applied before the
         epilogue.  ``emit_norm`` = (weight, eps) with EPI_ADD_F32 returns the ``NormedActivation`` of the
@@ -1891,7 +1897,29 @@ class CudaOps:
         return y, res_out
 
     def linear_add_tanh_norm(self, x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor, norm, scale: torch.Tensor) -> torch.Tensor:
-        """residual += scale * (x @ w^T), and the norm of the new residual."""
+        """residual += scale * (x @ w^T), and the norm of the new residual.  In 16-bit steps of few tokens both happen in the
+        product's epilogue."""
+        M, K = x.shape
+        if x.dtype == torch.bfloat16 and self.fuses_next_norm and M <= self.FUSED_NORM_MAX_TOKENS and M <= 64 and K % 8 == 0 and K >= 64:
+            alpha, weight, bias = norm
+            for name, t in (("residual", residual), ("scale", scale), ("norm weight", weight), ("norm bias", bias)):
+                self._want(t, name, torch.float32)
+            self._want(x, "x")
+            self._want(w, "w", x.dtype)
+            N = w.shape[0]
+            if tuple(residual.shape) != (M, N) or w.shape[1] != K or any(t.numel() != N for t in (scale, weight, bias)):
+                raise KernelError("linear_add_tanh_norm: shapes do not fit")
+            y = self.empty((M, N), x.dtype)
+            rc = -2
+            if M <= 8 and self.small_products:
+                rc = self.lib.ptl_gemm_small_tanh_norm_bf16(_p(residual), _p(x), _p(w), M, N, K, _p(scale), _p(weight), _p(bias), float(alpha),
+                                                            _p(y), self._stream())
+            if rc == -2:
+                rc = self.lib.ptl_gemm_tc_tanh_norm_bf16(_p(residual), _p(x), _p(w), M, N, K, _p(self._tc_status_word()), _p(scale), _p(weight),
+                                                         _p(bias), float(alpha), _p(y), self._stream())
+            if rc != -2:
+                self._check(rc)
+                return y
         return self.add_tanh_norm(self.linear(x, w), residual, norm, scale=scale, dtype=x.dtype)[0]
 
     def combine_experts_tanh_norm(self, rows: "ExpertRows", shared: Optional[torch.Tensor], residual: torch.Tensor, norm,
@@ -1900,7 +1928,11 @@ class CudaOps:
         return self.add_tanh_norm(shared, residual, norm, scale=scale, dtype=rows.x.dtype, experts=rows)[0]
 
     def linear_relu2(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-        """max(x @ w^T, 0)^2."""
+        """max(x @ w^T, 0)^2, in the epilogue of this library's 16-bit product."""
+        if x.dtype == torch.bfloat16 and not self.library_product(x.shape[0], w.shape[0], x.shape[1], self.EPI_BF16):
+            y = self.gemm_tc(x, w, self.EPI_RELU2)
+            if y is not None:
+                return y
         y = self.linear(x, w)
         self._check(getattr(self.lib, "ptl_relu2" + _suffix(y.dtype))(_p(y), y.numel(), self._stream()))
         return y
@@ -1924,6 +1956,11 @@ class CudaOps:
                 matmul.allow_bf16_reduced_precision_reduction = before
         plane = -(-T * N // 8) * 8                 # every result starts on a 16-byte boundary
         out = self.empty((n, plane), x.dtype)[:, :T * N].unflatten(1, (T, N))
+        if x.dtype == torch.bfloat16 and T <= 8 and self.small_products and K >= 64:
+            rc = self.lib.ptl_gemm_small_each_bf16(_p(out), plane, _p(x), T * K, _p(w), N * K, n, T, N, K, self._stream())
+            if rc != -2:
+                self._check(rc)
+                return out
         for i in range(n):
             if x.dtype == torch.float32:
                 self._check(self.lib.ptl_gemm_simt_f32(_p(out[i]), _p(x[i]), _p(w[i]), T, N, K, K, K, N, 0, self._stream()))
