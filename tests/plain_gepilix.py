@@ -335,7 +335,7 @@ def tensor_shapes(cfg: dict, rank: int = 16) -> Dict[str, tuple]:
 def random_weights(cfg: dict, seed: int, dtype=torch.float32, rank: int = 16) -> Dict[str, torch.Tensor]:
     """Weights drawn so that no mechanism drowns: matrices N(0, 1.5^2 / fan_in), scores of a few units, decays from
     near one to near zero, router logits that spread.  In 16 bits scores are smaller (a score s carries a rounding error
-    of about |s| * 2^-8)."""
+    of about |s| * 2^-8), and so are the routed experts' outputs (a router's close call that falls the other way swaps them)."""
     gentle = dtype != torch.float32
     gen = torch.Generator().manual_seed(seed)
     rand = lambda *s: torch.randn(*s, generator=gen, dtype=torch.float32)
@@ -374,6 +374,8 @@ def random_weights(cfg: dict, seed: int, dtype=torch.float32, rank: int = 16) ->
             t = rand(*shape) * ((1.5 if gentle else 3.0) / math.sqrt(shape[-1]))
         else:
             t = rand(*shape) * (1.5 / math.sqrt(shape[-1]))
+            if gentle and last == "down" and parts[-2].startswith("e"):
+                t *= 0.25
         out[name] = t.to(dtype)
     return out
 
