@@ -8,26 +8,27 @@
 //
 // q_scale and k_scale multiply queries and keys.  q, k and v are rows of T elements with a pitch each; head h's q and k start
 // at (h / per_qk) * d, its v at h * dv.  z is float32 [T, H*d] before the bias, dt float32 [T, H].
-// A block owns 32 columns of one head's state for one request and walks the request's
-// tokens of this step in order.  The 32 lanes of a warp are the 32 columns; each of the 8 warps holds
-// every eighth packet of four of the d rows in registers (as pairs: the products and sums are the two-wide float32
+// A block owns COLS (32 or 16) columns of one head's state for one request and walks the request's
+// tokens of this step in order.  Neighbouring threads are neighbouring columns; each of the 256 / COLS groups of them holds
+// every eighth (sixteenth) packet of four of the d rows in registers (as pairs: the products and sums are the two-wide float32
 // instructions, which round each half like the scalar forms), so the q, k and decay values a warp needs
-// are the same for all its lanes: one shared-memory wavefront per packet.  (With 8 lanes per column
+// are the same for all its lanes (for each half of them): one shared-memory wavefront per packet.  16 columns are taken
+// where blocks of 32 would leave half the SMs empty (measured at 2,048 tokens of one request: 64 blocks of 32 columns 358 us, 128 of
+// 16 274 us; from about a block per SM on, staging every token twice as often costs more than it brings).  (With 8 lanes per column
 // and the rows spread over the lanes the kernel was bound by shared-memory bandwidth, 437 wavefronts a
-// token.)  Nothing in the walk waits on a shuffle; the warps' partial read-outs of a batch meet in
+// token.)  Nothing in the walk waits on a shuffle; the groups' partial read-outs of a batch meet in
 // shared memory.  Tokens come through shared memory in batches (q scaled, decay worked out while
 // staging; the next batch's values are requested before the walk over this one).  What a token adds to its own read-out
 // beside S (the bonus's sum over q u k, or D) is one number per token and head times v, added where the parts meet.  The state of a
 // request is read from its slot unless the portion starts at position 0 and written back at the end.
-// Everything after the loads is float32; a token's result does not depend on how the request was cut
-// into steps or on what else the step holds.
+// Everything after the loads is float32; a state does not depend on how the request was cut into steps or on what else the
+// step holds, a read-out only through the grouping of its sum (16 or 32 columns).
 #include "common.cuh"
 
 namespace ptl {
 
-constexpr int kGlaCols = 32;      // columns of the state per block
-constexpr int kGlaLanes = 8;      // threads per column (one in each warp)
-constexpr int kGlaThreads = kGlaCols * kGlaLanes;
+constexpr int kGlaThreads = 256;
+constexpr int kGlaNarrowBlocks = 74;      // up to so many blocks of 32 columns (half the SMs), blocks take 16
 
 enum GlaForm { kGlaSigmoid = 0, kGlaFixed = 1, kGlaBonus = 2, kGlaStep = 3 };
 
@@ -52,14 +53,15 @@ __device__ __forceinline__ float gla_softplus(float x) { return x > 20.f ? x : l
 // exp(x), x <= 0, rounded once near 1: a decay of almost 1 acts a thousand times over, and any lean of its last bit with it
 __device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
 
-template <typename T, int RPL, int TB, int FORM>   // RPL rows per lane (d <= 8 * RPL), TB tokens per batch
+template <typename T, int COLS, int RPL, int TB, int FORM>   // RPL rows per thread (d <= 256 / COLS * RPL), TB tokens per batch
 __global__ void __launch_bounds__(kGlaThreads)
 gla_scan_kernel(const GlaArgs p) {
-  constexpr int DP = kGlaLanes * RPL;
+  constexpr int kGroups = kGlaThreads / COLS;      // threads per column
+  constexpr int DP = kGroups * RPL;
   constexpr bool kChannel = FORM == kGlaSigmoid || FORM == kGlaBonus;      // a decay per channel
   __shared__ __align__(16) float s_q[TB][DP], s_k[TB][DP], s_a[kChannel ? TB : 1][kChannel ? DP : 4];
-  __shared__ float s_v[TB][kGlaCols];
-  __shared__ float s_part[TB][kGlaLanes][kGlaCols];        // a warp's part of a token's read-out, per column
+  __shared__ float s_v[TB][COLS];
+  __shared__ float s_part[TB][kGroups][COLS];              // a group's part of a token's read-out, per column
   __shared__ float s_step[2][TB], s_dec[2][TB];            // step form: a token's step size and decay, this batch's and the next's
   __shared__ float s_own[TB];                              // bonus form: sum of q u k
   pdl_wait();
@@ -70,11 +72,12 @@ gla_scan_kernel(const GlaArgs p) {
   if (t1 <= t0 || slot < 0) return;
   const int H = p.H, d = p.d, dv = p.dv;
   const int tid = threadIdx.x;
-  const int col = tid & 31, lane8 = tid >> 5;              // column = lane; lane8: which eighth of the rows = the warp
-  const int e = blockIdx.x * kGlaCols + col;
+  const int col = tid % COLS, grp = tid / COLS;            // grp: which share of the rows
+  const int lane = tid & 31, warp = tid >> 5;
+  const int e = blockIdx.x * COLS + col;
   const bool live = e < dv;
-  // rows of this warp: packets of four, packet m of the warp being packet m * 8 + lane8 of the column
-  auto row_of = [&](int i) { return ((i >> 2) * kGlaLanes + lane8) * 4 + (i & 3); };
+  // rows of this thread: packets of four, its packet m being packet m * kGroups + grp of the column
+  auto row_of = [&](int i) { return ((i >> 2) * kGroups + grp) * 4 + (i & 3); };
   float* st = p.state + (((size_t)slot * H + h) * d) * dv;
   float2 S[RPL / 2];
   const bool fresh = p.positions[t0] == 0;
@@ -85,13 +88,13 @@ gla_scan_kernel(const GlaArgs p) {
   }
   const T* qp = reinterpret_cast<const T*>(p.q) + (size_t)(h / p.per_qk) * d;
   const T* kp = reinterpret_cast<const T*>(p.k) + (size_t)(h / p.per_qk) * d;
-  const T* vp = reinterpret_cast<const T*>(p.v) + (size_t)h * dv + blockIdx.x * kGlaCols;
-  const int vcols = min(kGlaCols, dv - blockIdx.x * kGlaCols);
+  const T* vp = reinterpret_cast<const T*>(p.v) + (size_t)h * dv + blockIdx.x * COLS;
+  const int vcols = min(COLS, dv - blockIdx.x * COLS);
 
   // A thread fetches the same column c of q, k and z for tokens j0, j0 + step, ...: the next batch's values are
   // requested before the walk over this batch and kept as fetched; they are converted (and the decay worked out)
   // when they go to shared memory, after the walk.
-  constexpr int NE = TB * DP / kGlaThreads, NV = (TB * kGlaCols + kGlaThreads - 1) / kGlaThreads;
+  constexpr int NE = TB * DP / kGlaThreads, NV = (TB * COLS + kGlaThreads - 1) / kGlaThreads;
   constexpr int kTokStep = kGlaThreads / DP > 0 ? kGlaThreads / DP : 1;
   static_assert(kGlaThreads % DP == 0 && NE * kTokStep == TB, "a thread's column must not change between its turns");
   const int c_mine = tid % DP, j_mine = tid / DP;
@@ -101,7 +104,7 @@ gla_scan_kernel(const GlaArgs p) {
   float bonus[(DP + 31) / 32];
   if constexpr (FORM == kGlaBonus) {
 #pragma unroll
-    for (int i = 0; i < (DP + 31) / 32; ++i) bonus[i] = col + 32 * i < d ? p.extra[h * d + col + 32 * i] : 0.f;
+    for (int i = 0; i < (DP + 31) / 32; ++i) bonus[i] = lane + 32 * i < d ? p.extra[h * d + lane + 32 * i] : 0.f;
   }
   T rq[NE], rk[NE], rv[NV];
   float rz[NE], rdt = 0.f;
@@ -119,7 +122,7 @@ gla_scan_kernel(const GlaArgs p) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int idx = tid + i * kGlaThreads;
-      const int j = idx / kGlaCols, c = idx % kGlaCols;
+      const int j = idx / COLS, c = idx % COLS;
       rv[i] = (j < nt && c < vcols) ? vp[(size_t)(tb + j) * p.v_ld + c] : from_f32<T>(0.f);
     }
     if (FORM == kGlaStep && tid < nt) rdt = p.dt[(size_t)(tb + tid) * H + h];
@@ -138,7 +141,7 @@ gla_scan_kernel(const GlaArgs p) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int idx = tid + i * kGlaThreads;
-      if (idx < TB * kGlaCols) s_v[idx / kGlaCols][idx % kGlaCols] = to_f32(rv[i]);
+      if (idx < TB * COLS) s_v[idx / COLS][idx % COLS] = to_f32(rv[i]);
     }
   };
   fetch(t0);
@@ -155,12 +158,12 @@ gla_scan_kernel(const GlaArgs p) {
     __syncthreads();
     if (tb + TB < t1) fetch(tb + TB);
     if constexpr (FORM == kGlaBonus) {     // read where the parts meet, behind the walk's barrier
-      for (int j = lane8; j < nt; j += kGlaLanes) {
+      for (int j = warp; j < nt; j += kGlaThreads / 32) {
         float s = 0.f;
 #pragma unroll
-        for (int i = 0; i < (DP + 31) / 32; ++i) s = fmaf(s_q[j][col + 32 * i] * s_k[j][col + 32 * i], bonus[i], s);
+        for (int i = 0; i < (DP + 31) / 32; ++i) s = fmaf(s_q[j][lane + 32 * i] * s_k[j][lane + 32 * i], bonus[i], s);
         s = warp_sum(s);
-        if (col == 0) s_own[j] = s;
+        if (lane == 0) s_own[j] = s;
       }
     }
     auto token = [&](int j) {
@@ -193,7 +196,7 @@ gla_scan_kernel(const GlaArgs p) {
           acc1 = __ffma2_rn(q1, S1, acc1);
         }
       }
-      s_part[j][lane8][col] = (acc0.x + acc0.y) + (acc1.x + acc1.y);
+      s_part[j][grp][col] = (acc0.x + acc0.y) + (acc1.x + acc1.y);
     };
     if (nt == TB) {
 #pragma unroll 4
@@ -202,15 +205,15 @@ gla_scan_kernel(const GlaArgs p) {
       for (int j = 0; j < nt; ++j) token(j);
     }
     __syncthreads();
-    // the warps' parts of every read-out of the batch, added in the order of the warps
-    for (int idx = tid; idx < nt * kGlaCols; idx += kGlaThreads) {
-      const int j = idx / kGlaCols, c = idx % kGlaCols;
+    // the groups' parts of every read-out of the batch, added in the order of the groups
+    for (int idx = tid; idx < nt * COLS; idx += kGlaThreads) {
+      const int j = idx / COLS, c = idx % COLS;
       float sum = 0.f;
 #pragma unroll
-      for (int w = 0; w < kGlaLanes; ++w) sum += s_part[j][w][c];
+      for (int w = 0; w < kGroups; ++w) sum += s_part[j][w][c];
       if constexpr (FORM == kGlaBonus) sum = fmaf(s_own[j], s_v[j][c], sum);
       if constexpr (FORM == kGlaStep) sum = fmaf(skip, s_v[j][c], sum);
-      if (c < vcols) p.out[(size_t)(tb + j) * H * dv + (size_t)h * dv + blockIdx.x * kGlaCols + c] = sum;
+      if (c < vcols) p.out[(size_t)(tb + j) * H * dv + (size_t)h * dv + blockIdx.x * COLS + c] = sum;
     }
   }
   if (live) {
@@ -227,12 +230,14 @@ int gla_launch(const char* what, const GlaArgs& p, int requests, void* stream) {
   PTL_REQUIRE(p.q_ld >= p.H / p.per_qk * p.d && p.k_ld >= p.H / p.per_qk * p.d && p.v_ld >= p.H * p.dv, "%s: rows are too short", what);
   PTL_REQUIRE(p.H <= 65535 && requests <= 65535, "%s: too many heads or requests", what);
   if (requests == 0) return 0;
-  const dim3 grid((p.dv + kGlaCols - 1) / kGlaCols, p.H, requests), block(kGlaThreads);
-#define PTL_GLA_LAUNCH(RPL, TB) return launch_kernel(what, gla_scan_kernel<T, RPL, TB, FORM>, grid, block, 0, as_stream(stream), p)
-  if (p.d <= 32) PTL_GLA_LAUNCH(4, 16);
-  if (p.d <= 64) PTL_GLA_LAUNCH(8, 16);
-  if (p.d <= 128) PTL_GLA_LAUNCH(16, 16);
-  PTL_GLA_LAUNCH(32, 8);
+#define PTL_GLA_LAUNCH(COLS, RPL, TB)                                                                                        \
+  return launch_kernel(what, gla_scan_kernel<T, COLS, RPL, TB, FORM>, dim3((p.dv + COLS - 1) / COLS, p.H, requests),           \
+                       dim3(kGlaThreads), 0, as_stream(stream), p)
+  if (p.d <= 32) PTL_GLA_LAUNCH(32, 4, 16);
+  const bool narrow = (long long)((p.dv + 31) / 32) * p.H * requests <= kGlaNarrowBlocks;
+  if (p.d <= 64) { if (narrow) PTL_GLA_LAUNCH(16, 4, 16); PTL_GLA_LAUNCH(32, 8, 16); }
+  if (p.d <= 128) { if (narrow) PTL_GLA_LAUNCH(16, 8, 16); PTL_GLA_LAUNCH(32, 16, 16); }
+  PTL_GLA_LAUNCH(32, 32, 8);
 #undef PTL_GLA_LAUNCH
 }
 

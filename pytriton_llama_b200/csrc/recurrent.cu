@@ -502,6 +502,55 @@ gated_head_norm_kernel(T* __restrict__ out, int out_ld, int column, const float*
   }
 }
 
+template <typename T>
+__device__ __forceinline__ float4 load_four(const T* p) {
+  if constexpr (sizeof(T) == 4) {
+    return *reinterpret_cast<const float4*>(p);
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store_four(T* p, float4 v) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = v;
+  } else {
+    uint2 raw;
+    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = raw;
+  }
+}
+
+// The same for heads of 4 * LPH entries (LPH lanes of four neighbours a head) whose rows start on packets.
+template <typename T, int LPH>
+__global__ void __launch_bounds__(256)
+gated_head_norm_packets_kernel(T* __restrict__ out, int out_ld, int column, const float* __restrict__ o, const float* __restrict__ w,
+                               float eps, const T* __restrict__ gate, int gate_ld, int gate_column, int tokens, int heads, float scale,
+                               int sigmoid_gate, int weight_per_head) {
+  constexpr int DV = 4 * LPH;
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t item = ((size_t)blockIdx.x * 256 + threadIdx.x) / LPH;
+  const int e = (threadIdx.x % LPH) * 4;
+  const bool live = item < (size_t)tokens * heads;
+  const int t = live ? (int)(item / heads) : 0, h = live ? (int)(item % heads) : 0;
+  const float4 x = *reinterpret_cast<const float4*>(o + ((size_t)t * heads + h) * DV + e);
+  const float4 g = load_four(gate + (size_t)t * gate_ld + gate_column + h * DV + e);
+  const float4 wv = *reinterpret_cast<const float4*>((weight_per_head ? w + (size_t)h * DV : w) + e);
+  float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+#pragma unroll
+  for (int k = LPH / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+  const float f = scale / sqrtf(ss / (float)DV + eps);
+  auto act = [&](float v) { return sigmoid_gate ? 1.0f / (1.0f + expf(-v)) : silu_f32(v); };
+  if (live)
+    store_four(out + (size_t)t * out_ld + column + h * DV + e,
+               make_float4(x.x * f * wv.x * act(g.x), x.y * f * wv.y * act(g.y), x.z * f * wv.z * act(g.z), x.w * f * wv.w * act(g.w)));
+}
+
 // ------------------------------------------------------------------ output gate, then a norm in equal parts
 // With x = o * silu(gate):  out[t, column + e] = x[e] / sqrt(mean over e's part of x^2 + eps) * w[e] * scale, the row being cut
 // into `groups` parts of `len`.  One block per (token, part); rows of whole packets keep their x in registers (NP packets
@@ -526,17 +575,8 @@ gated_group_norm_kernel(T* __restrict__ out, int out_ld, int column, const float
       x[n] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (i < len) {
         x[n] = *reinterpret_cast<const float4*>(src + i);
-        float gv[4];
-        if constexpr (sizeof(T) == 4) {
-          const float4 v = *reinterpret_cast<const float4*>(g + i);
-          gv[0] = v.x; gv[1] = v.y; gv[2] = v.z; gv[3] = v.w;
-        } else {
-          const uint2 raw = *reinterpret_cast<const uint2*>(g + i);
-          const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-          const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-          gv[0] = a.x; gv[1] = a.y; gv[2] = b.x; gv[3] = b.y;
-        }
-        x[n].x *= silu_f32(gv[0]); x[n].y *= silu_f32(gv[1]); x[n].z *= silu_f32(gv[2]); x[n].w *= silu_f32(gv[3]);
+        const float4 gv = load_four(g + i);
+        x[n].x *= silu_f32(gv.x); x[n].y *= silu_f32(gv.y); x[n].z *= silu_f32(gv.z); x[n].w *= silu_f32(gv.w);
         ss = fmaf(x[n].x, x[n].x, fmaf(x[n].y, x[n].y, fmaf(x[n].z, x[n].z, fmaf(x[n].w, x[n].w, ss))));
       }
     }
@@ -546,15 +586,7 @@ gated_group_norm_kernel(T* __restrict__ out, int out_ld, int column, const float
       const int i = (n * 256 + threadIdx.x) * 4;
       if (i >= len) continue;
       const float4 wv = *reinterpret_cast<const float4*>(w + at + i);
-      const float4 y = make_float4(x[n].x * f * wv.x, x[n].y * f * wv.y, x[n].z * f * wv.z, x[n].w * f * wv.w);
-      if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(dst + i) = y;
-      } else {
-        uint2 raw;
-        *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(y.x, y.y);
-        *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(y.z, y.w);
-        *reinterpret_cast<uint2*>(dst + i) = raw;
-      }
+      store_four(dst + i, make_float4(x[n].x * f * wv.x, x[n].y * f * wv.y, x[n].z * f * wv.z, x[n].w * f * wv.w));
     }
   } else {
     for (int i = threadIdx.x; i < len; i += 256) {
@@ -674,6 +706,17 @@ int gated_head_norm(void* out, int out_ld, int column, const float* o, const flo
               tokens, heads, dv);
   if (tokens == 0) return 0;
   const size_t items = (size_t)tokens * heads;
+  const T* g = (const T*)gate + gate_column;
+  T* dst = (T*)out + column;
+  const bool packets = gate_ld % 4 == 0 && out_ld % 4 == 0 && aligned16(o) && aligned16(w) && ((uintptr_t)g % (4 * sizeof(T))) == 0 &&
+                       ((uintptr_t)dst % (4 * sizeof(T))) == 0;
+#define PTL_GHN(LPH) return launch_kernel("gated_head_norm", gated_head_norm_packets_kernel<T, LPH>,                              \
+    dim3((unsigned)((items * LPH + 255) / 256)), dim3(256), 0, as_stream(stream), (T*)out, out_ld, column, o, w, eps,              \
+    (const T*)gate, gate_ld, gate_column, tokens, heads, scale, sigmoid_gate, weight_per_head)
+  if (packets && dv == 32) PTL_GHN(8);
+  if (packets && dv == 64) PTL_GHN(16);
+  if (packets && dv == 128) PTL_GHN(32);
+#undef PTL_GHN
   return launch_kernel("gated_head_norm", gated_head_norm_kernel<T>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0,
                        as_stream(stream), (T*)out, out_ld, column, o, w, eps, (const T*)gate, gate_ld, gate_column, tokens, heads,
                        dv, scale, sigmoid_gate, weight_per_head);
