@@ -33,12 +33,23 @@ struct LruArgs {
   float scale;
 };
 
-__device__ __forceinline__ float lru_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float lru_gelu(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// FAST (16-bit inputs): the fast exponential and quotient, off by about |z| * 2^-23, beside inputs rounded to 2^-9.  The decay
+// itself is always worked out in full.
+template <bool FAST>
+__device__ __forceinline__ float lru_sigmoid(float z) {
+  return FAST ? __fdividef(1.0f, 1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+}
+// 0.5 z (1 + tanh(v)) = z sigmoid(2 v), v = sqrt(2/pi) (z + 0.044715 z^3)
+template <bool FAST>
+__device__ __forceinline__ float lru_gelu(float z) {
+  const float v = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return FAST ? z * lru_sigmoid<true>(2.0f * v) : 0.5f * z * (1.0f + tanhf(v));
+}
 // a - 1 and what enters the state
+template <bool FAST>
 __device__ __forceinline__ void lru_gates(float zr, float zi, float rate, float u, float& e, float& add) {
-  e = expm1f(-rate * lru_sigmoid(zr));
-  add = sqrtf(-e * (2.0f + e)) * lru_sigmoid(zi) * u;
+  e = expm1f(-rate * lru_sigmoid<FAST>(zr));
+  add = sqrtf(-e * (2.0f + e)) * lru_sigmoid<FAST>(zi) * u;
 }
 // a S + add
 __device__ __forceinline__ float lru_step(float e, float S, float add) { return S + fmaf(e, S, add); }
@@ -83,9 +94,9 @@ gated_lru_scan_kernel(const float* __restrict__ z, long long z_block, long long 
     float E = 0.f, B = 0.f;
 #pragma unroll
     for (int k = 0; k < kLruTokens; ++k) {
-      lru_gates(zr[k] + br, zi[k] + bi, rate, to_f32(ru[k]), e[k], add[k]);
+      lru_gates<sizeof(T) == 2>(zr[k] + br, zi[k] + bi, rate, to_f32(ru[k]), e[k], add[k]);
       if (first + k >= hi) { e[k] = 0.f; add[k] = 0.f; }       // past the end: nothing changes
-      g[k] = lru_gelu(to_f32(ry[k]) + by) * p.scale;
+      g[k] = lru_gelu<sizeof(T) == 2>(to_f32(ry[k]) + by) * p.scale;
       E = lru_step(e[k], E, e[k]);
       B = lru_step(e[k], B, add[k]);
     }
@@ -158,11 +169,11 @@ gated_lru_single_kernel(const __nv_bfloat16* __restrict__ w, int s, const int* _
   const int r = tok_req[lane];
   if (r < 0 || p.state_slot[r] < 0) return;
   float less, add;
-  lru_gates(zr + p.gate_bias[c], zi + p.gate_bias[p.n + c], p.rate[c], __bfloat162float(ub[(size_t)lane * p.n + e]), less, add);
+  lru_gates<true>(zr + p.gate_bias[c], zi + p.gate_bias[p.n + c], p.rate[c], __bfloat162float(ub[(size_t)lane * p.n + e]), less, add);
   float* st = p.state + (size_t)p.state_slot[r] * p.n + c;
   const float S = lru_step(less, p.positions[lane] == 0 ? 0.f : *st, add);
   *st = S;
-  const float g = lru_gelu(__bfloat162float(((const __nv_bfloat16*)p.y)[(size_t)lane * p.y_ld + c]) + p.y_bias[c]) * p.scale;
+  const float g = lru_gelu<true>(__bfloat162float(((const __nv_bfloat16*)p.y)[(size_t)lane * p.y_ld + c]) + p.y_bias[c]) * p.scale;
   ((__nv_bfloat16*)p.out)[(size_t)lane * p.out_ld + p.column + c] = __float2bfloat16_rn(S * g);
 }
 
