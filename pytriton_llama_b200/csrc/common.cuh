@@ -70,6 +70,9 @@ template <typename T> __device__ __forceinline__ void store16(T* p, const Vec16<
   *reinterpret_cast<decltype(v.raw)*>(p) = v.raw;
 }
 
+// exp(x), x <= 0, rounded once near 1: a decay of almost 1 acts a thousand times over, and any lean of its last bit with it.
+__device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
+
 // ---------------------------------------------------------------- reductions
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

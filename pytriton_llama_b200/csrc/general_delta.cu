@@ -200,7 +200,8 @@ int general_delta_scan(float* out, const void* proj, int ld, const float* a_pre,
 #undef PTL_GD
 }
 
-// z[t, c] = sum_j w2[c, j] * tanh(x[t, column + j]), float32 throughout.  Every result is one chain of fused
+// z[t, c] = sum_j w2[c, j] * tanh(x[t, column + j]), float32 throughout; with `decay_bias` the result is the decay
+// exp(-exp(z + decay_bias[c])) instead.  Every result is one chain of fused
 // multiply-adds, j ascending, whatever the tile it falls into, so a token's row has the same bits in a prompt
 // portion and alone.  A block takes kLtTokens tokens and kLtCols columns: the inner inputs' tanh and a slab of w2
 // (kLtRank values of j at a time, transposed so that neighbouring threads read neighbouring words) go through shared
@@ -209,7 +210,7 @@ constexpr int kLtTokens = 16, kLtCols = 128, kLtRank = 32;
 
 __global__ void __launch_bounds__(kLtCols)
 lowrank_tanh_linear_kernel(float* __restrict__ z, const float* __restrict__ x, int tokens, int x_ld, int column, int rank,
-                           const float* __restrict__ w2, int n) {
+                           const float* __restrict__ w2, int n, const float* __restrict__ decay_bias) {
   __shared__ __align__(16) float s_hid[kLtRank][kLtTokens];      // tanh of the inner inputs, tokens side by side
   __shared__ float s_w[kLtRank][kLtCols + 1];
   pdl_wait();
@@ -245,23 +246,24 @@ lowrank_tanh_linear_kernel(float* __restrict__ z, const float* __restrict__ x, i
     }
   }
   if (c < n) {
+    const float bias = decay_bias ? decay_bias[c] : 0.f;
 #pragma unroll
     for (int t = 0; t < kLtTokens; ++t)
-      if (t0 + t < tokens) z[(size_t)(t0 + t) * n + c] = acc[t];
+      if (t0 + t < tokens) z[(size_t)(t0 + t) * n + c] = decay_bias ? decay_exp(-expf(acc[t] + bias)) : acc[t];
   }
 }
 
 }  // namespace ptl
 
 PTL_EXPORT int ptl_lowrank_tanh_linear(float* z, const float* x, int tokens, int x_ld, int column, int rank, const float* w2, int n,
-                                       void* stream) {
+                                       const float* decay_bias, void* stream) {
   PTL_REQUIRE(tokens >= 0 && rank > 0 && n > 0 && column >= 0 && column + rank <= x_ld,
               "lowrank_tanh_linear: bad sizes rank=%d n=%d column=%d ld=%d", rank, n, column, x_ld);
   if (tokens == 0) return 0;
   const dim3 grid((n + ptl::kLtCols - 1) / ptl::kLtCols, (tokens + ptl::kLtTokens - 1) / ptl::kLtTokens);
   PTL_REQUIRE(grid.y <= 65535, "lowrank_tanh_linear: %d tokens in one call", tokens);
   return ptl::launch_kernel("lowrank_tanh_linear", ptl::lowrank_tanh_linear_kernel, grid, dim3(ptl::kLtCols), 0,
-                            ptl::as_stream(stream), z, x, tokens, x_ld, column, rank, w2, n);
+                            ptl::as_stream(stream), z, x, tokens, x_ld, column, rank, w2, n, decay_bias);
 }
 
 #define PTL_GENERAL_DELTA(SUFFIX, TYPE)                                                                                          \

@@ -2,12 +2,12 @@
 //
 //   sigmoid  S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t,  a_t = sigmoid(z_t + b)^(1/tau) = exp(logsigmoid(z_t + b) / tau)
 //   fixed    the same with one fixed decay per head (retention)
-//   bonus    o_t = (S + diag(u) k_t v_t^T)^T q_t, then S <- diag(a_t) S + k_t v_t^T, a_t = exp(-exp(z_t + b)) (RWKV)
+//   bonus    o_t = (S + diag(u) k_t v_t^T)^T q_t, then S <- diag(a_t) S + k_t v_t^T, the decays a_t given (RWKV)
 //   step     S <- exp(-rate_h s_t) S + s_t k_t v_t^T, o_t = S^T q_t + D_h v_t, s_t = softplus(dt_t + dt_bias_h) per head and
 //            token (state space), q and k shared by groups of heads
 //
 // q_scale and k_scale multiply queries and keys.  q, k and v are rows of T elements with a pitch each; head h's q and k start
-// at (h / per_qk) * d, its v at h * dv.  z is float32 [T, H*d] before the bias, dt float32 [T, H].
+// at (h / per_qk) * d, its v at h * dv.  z is float32 [T, H*d], before the bias or the decay itself, dt float32 [T, H].
 // A block owns COLS (32 or 16) columns of one head's state for one request and walks the request's
 // tokens of this step in order.  Neighbouring threads are neighbouring columns; each of the 256 / COLS groups of them holds
 // every eighth (sixteenth) packet of four of the d rows in registers (as pairs: the products and sums are the two-wide float32
@@ -36,7 +36,7 @@ struct GlaArgs {
   float* out;                     // [T, H*dv]
   const void *q, *k, *v;
   int q_ld, k_ld, v_ld, per_qk;
-  const float *z, *bias;          // sigmoid, bonus
+  const float *z, *bias;          // sigmoid; bonus: z is the decay, no bias
   float inv_tau;                  // sigmoid
   const float* head;              // fixed: the decay; step: the rate
   const float *dt, *dt_bias;      // step
@@ -49,9 +49,6 @@ struct GlaArgs {
 
 __device__ __forceinline__ float log_sigmoid_f32(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gla_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-
-// exp(x), x <= 0, rounded once near 1: a decay of almost 1 acts a thousand times over, and any lean of its last bit with it
-__device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
 
 template <typename T, int COLS, int RPL, int TB, int FORM>   // RPL rows per thread (d <= 256 / COLS * RPL), TB tokens per batch
 __global__ void __launch_bounds__(kGlaThreads)
@@ -98,7 +95,7 @@ gla_scan_kernel(const GlaArgs p) {
   constexpr int kTokStep = kGlaThreads / DP > 0 ? kGlaThreads / DP : 1;
   static_assert(kGlaThreads % DP == 0 && NE * kTokStep == TB, "a thread's column must not change between its turns");
   const int c_mine = tid % DP, j_mine = tid / DP;
-  const float b_mine = (kChannel && c_mine < d) ? p.bias[h * d + c_mine] : 0.f;
+  const float b_mine = (FORM == kGlaSigmoid && c_mine < d) ? p.bias[h * d + c_mine] : 0.f;
   const float head_h = kChannel ? 0.f : p.head[h];         // the fixed decay, or the step form's rate
   const float dt_bias = FORM == kGlaStep ? p.dt_bias[h] : 0.f, skip = FORM == kGlaStep ? p.extra[h] : 0.f;
   float bonus[(DP + 31) / 32];
@@ -136,7 +133,7 @@ gla_scan_kernel(const GlaArgs p) {
       if constexpr (FORM == kGlaStep) k *= s_step[buf][j];
       s_k[j][c_mine] = k;
       if constexpr (FORM == kGlaSigmoid) s_a[j][c_mine] = c_mine < d ? expf(log_sigmoid_f32(rz[i] + b_mine) * p.inv_tau) : 0.f;
-      if constexpr (FORM == kGlaBonus) s_a[j][c_mine] = c_mine < d ? decay_exp(-expf(rz[i] + b_mine)) : 0.f;
+      if constexpr (FORM == kGlaBonus) s_a[j][c_mine] = rz[i];
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -258,13 +255,13 @@ int gla_scan(float* out, const void* proj, int ld, const float* z, const float* 
 
 // rkv: the rows of r, k and v are `plane` elements apart, each [T, H*d].
 template <typename T>
-int wkv_scan(float* out, const void* rkv, long long plane, const float* z, const float* bias, const float* u, float* state,
+int wkv_scan(float* out, const void* rkv, long long plane, const float* decay, const float* u, float* state,
              const int* q_start, const int* positions, const int* state_slot, int requests, int H, int d, void* stream) {
-  PTL_REQUIRE(z && bias && u && plane >= 0, "wkv_scan: missing operands");
+  PTL_REQUIRE(decay && u && plane >= 0, "wkv_scan: missing operands");
   const T* rows = (const T*)rkv;
   GlaArgs p{};
   p.out = out; p.q = rows; p.k = rows + plane; p.v = rows + 2 * plane; p.q_ld = p.k_ld = p.v_ld = H * d; p.per_qk = 1;
-  p.z = z; p.bias = bias; p.extra = u; p.state = state;
+  p.z = decay; p.extra = u; p.state = state;
   p.q_start = q_start; p.positions = positions; p.state_slot = state_slot; p.H = H; p.d = d; p.dv = d; p.q_scale = p.k_scale = 1.f;
   return gla_launch<T, kGlaBonus>("wkv_scan", p, requests, stream);
 }
@@ -294,10 +291,10 @@ int state_space_scan(float* out, const void* xbc, int ld, const float* dt, const
     return ptl::gla_scan<TYPE>(out, proj, ld, z, bias, inv_tau, state, q_start, positions, state_slot, requests, H, d, dv,       \
                                q_scale, head_decay, k_scale, stream);                                                           \
   }                                                                                                                             \
-  PTL_EXPORT int ptl_wkv_scan##SUFFIX(float* out, const void* rkv, long long plane, const float* z, const float* bias,           \
-                                      const float* u, float* state, const int* q_start, const int* positions,                   \
+  PTL_EXPORT int ptl_wkv_scan##SUFFIX(float* out, const void* rkv, long long plane, const float* decay, const float* u,          \
+                                      float* state, const int* q_start, const int* positions,                   \
                                       const int* state_slot, int requests, int H, int d, void* stream) {                        \
-    return ptl::wkv_scan<TYPE>(out, rkv, plane, z, bias, u, state, q_start, positions, state_slot, requests, H, d, stream);      \
+    return ptl::wkv_scan<TYPE>(out, rkv, plane, decay, u, state, q_start, positions, state_slot, requests, H, d, stream);      \
   }                                                                                                                             \
   PTL_EXPORT int ptl_state_space_scan##SUFFIX(float* out, const void* xbc, int ld, const float* dt, const float* dt_bias,        \
                                               const float* rate, const float* D, float* state, const int* q_start,              \

@@ -72,7 +72,7 @@ _SIGNATURES = {
     "ptl_head_linear": [_ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr],
     "ptl_gla_scan": [_ptr, _ptr, _c_int, _ptr, _ptr, _c_f, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr, _c_f,
                      _ptr],
-    "ptl_wkv_scan": [_ptr, _ptr, _c_ll, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr],
+    "ptl_wkv_scan": [_ptr, _ptr, _c_ll, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _ptr],
     "ptl_state_space_scan": [_ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _ptr],
     "ptl_gated_group_norm": [_ptr, _c_int, _c_int, _ptr, _ptr, _c_f, _ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _ptr],
     "ptl_gated_lru_scan": [_ptr, _c_int, _c_int, _ptr, _ptr, _c_ll, _c_ll, _c_int, _ptr, _ptr, _ptr, _c_int, _ptr, _ptr, _ptr, _ptr, _ptr,
@@ -205,7 +205,7 @@ def load_library() -> ctypes.CDLL:
     lib.ptl_moe_grouped_wide_bf16.restype = _c_int
     lib.ptl_pair_angles.argtypes = [_ptr, _ptr, _ptr, _c_int, _c_int, _c_f, _ptr]
     lib.ptl_pair_angles.restype = _c_int
-    lib.ptl_lowrank_tanh_linear.argtypes = [_ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr]
+    lib.ptl_lowrank_tanh_linear.argtypes = [_ptr, _ptr, _c_int, _c_int, _c_int, _c_int, _ptr, _c_int, _ptr, _ptr]
     lib.ptl_lowrank_tanh_linear.restype = _c_int
     lib.ptl_head_linear_few_bf16.argtypes = _SIGNATURES["ptl_head_linear"]
     lib.ptl_head_linear_few_bf16.restype = _c_int
@@ -1537,8 +1537,13 @@ class CudaOps:
         self._check(fn(_p(out), _p(x), x.numel(), float(pos_factor), float(neg_factor), self._stream()))
         return out
 
-    def lowrank_tanh_linear(self, x: torch.Tensor, column: int, w2: torch.Tensor) -> torch.Tensor:
-        """tanh(x[:, column:column + rank]) @ w2[n, rank]^T, float32 [T, n]."""
+    def lowrank_tanh_linear(self, x: torch.Tensor, column: int, w2: torch.Tensor, decay_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """z = tanh(x[:, column:column + rank]) @ w2[n, rank]^T, float32 [T, n]; with ``decay_bias`` float32 [n] the decay
+        exp(-exp(z + decay_bias))."""
+        if decay_bias is not None:
+            self._want(decay_bias, "decay bias", torch.float32)
+            if decay_bias.numel() != w2.shape[0]:
+                raise KernelError("lowrank_tanh_linear: one decay bias per column")
         self._want(x, "x", torch.float32)
         self._want(w2, "w2", torch.float32)
         n, rank = w2.shape
@@ -1546,7 +1551,7 @@ class CudaOps:
             raise KernelError("lowrank_tanh_linear: the inner inputs are the last columns of x")
         z = self.empty((x.shape[0], n), torch.float32)
         self._check(self.lib.ptl_lowrank_tanh_linear(_p(z), _p(x), x.shape[0], x.shape[1], int(column), rank, _p(w2), n,
-                                                     self._stream()))
+                                                     _p(decay_bias), self._stream()))
         return z
 
     def general_delta_scan(self, proj: torch.Tensor, aw: torch.Tensor, a_bias: torch.Tensor, z: torch.Tensor, w_bias: torch.Tensor,
@@ -1983,20 +1988,18 @@ class CudaOps:
             _p(ctx.state_slot), self._stream()))
         return out
 
-    def wkv_scan(self, rkvg: torch.Tensor, z: torch.Tensor, w_bias: torch.Tensor, u: torch.Tensor, state: torch.Tensor, ctx, H: int,
-                 d: int) -> torch.Tensor:
-        """The recurrence of ``parts/wkv.py``: rkvg [>= 3, T, H*d] (r, k, v, ...); z float32 [T, H*d], the decay's argument before
-        its bias; u float32 [H*d]; state float32 [slots, H, d, d]; returns the heads' read-outs, float32 [T, H*d]."""
+    def wkv_scan(self, rkvg: torch.Tensor, decay: torch.Tensor, u: torch.Tensor, state: torch.Tensor, ctx, H: int, d: int) -> torch.Tensor:
+        """The recurrence of ``parts/wkv.py``: rkvg [>= 3, T, H*d] (r, k, v, ...); decay float32 [T, H*d]; u float32 [H*d]; state float32 [slots, H, d, d]; returns the heads' read-outs, float32 [T, H*d]."""
         self._want(rkvg[0], "r")                  # (the planes may lie further apart than their size)
-        for name, t in (("z", z), ("w_bias", w_bias), ("u", u), ("state", state)):
+        for name, t in (("decay", decay), ("u", u), ("state", state)):
             self._want(t, name, torch.float32)
         n, T = H * d, rkvg.shape[1]
-        if rkvg.shape[0] < 3 or rkvg.shape[2] != n or tuple(z.shape) != (T, n) or w_bias.numel() != n or u.numel() != n or \
+        if rkvg.shape[0] < 3 or rkvg.shape[2] != n or tuple(decay.shape) != (T, n) or u.numel() != n or \
                 tuple(state.shape[1:]) != (H, d, d):
             raise KernelError("wkv_scan: shapes do not fit")
         out = self.empty((T, n), torch.float32)
         self._check(getattr(self.lib, "ptl_wkv_scan" + _suffix(rkvg.dtype))(
-            _p(out), _p(rkvg), rkvg.stride(0), _p(z), _p(w_bias), _p(u), _p(state), _p(ctx.q_start), _p(ctx.positions), _p(ctx.state_slot),
+            _p(out), _p(rkvg), rkvg.stride(0), _p(decay), _p(u), _p(state), _p(ctx.q_start), _p(ctx.positions), _p(ctx.state_slot),
             ctx.num_requests, H, d, self._stream()))
         return out
 

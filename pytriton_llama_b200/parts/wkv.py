@@ -65,8 +65,8 @@ class WKV(Part):
         H, d = self.heads, self.d
         mixes = ops.token_shift(x, self.mu, cache.states["last"], ctx)               # [5, T, hidden]
         rkvg = ops.linear_each(mixes[:4], self.w_rkvg)                                # [4, T, n]
-        z = ops.lowrank_tanh_linear(ops.linear(mixes[4], self.w_w1, out_dtype=torch.float32), 0, self.w_w2)     # before the bias
-        o = ops.wkv_scan(rkvg, z, self.w_bias, self.u, cache.states["S"], ctx, H, d)
+        decay = ops.lowrank_tanh_linear(ops.linear(mixes[4], self.w_w1, out_dtype=torch.float32), 0, self.w_w2, decay_bias=self.w_bias)
+        o = ops.wkv_scan(rkvg, decay, self.u, cache.states["S"], ctx, H, d)
         out = ops.empty((x.shape[0], H * d), self.rt.dtype)
         ops.gated_head_norm(o, self.norm_w, self.norm_eps, rkvg[3], 0, H, d, out, 0, 1.0, weight_per_head=True)
         return ops.linear(out, self.w_o) if tail is None else tail.product(out, self.w_o)

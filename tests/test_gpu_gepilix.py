@@ -230,11 +230,13 @@ def test_wkv_walk_with_its_bonus(ops, dtype, step, H, d):
     dt, ref = DTYPES[dtype], TorchOps()
     cd, cc, T = _both(step)
     n = H * d
-    rkvg, z = _rand(g, 4, T, n, scale=0.7).to(dt), _rand(g, T, n)
+    rkvg, inner, w2 = _rand(g, 4, T, n, scale=0.7).to(dt), _rand(g, T, 7), _rand(g, n, 7, scale=0.4)
     bias, u, state = torch.empty(n).uniform_(-9.0, 1.0, generator=g), _rand(g, n), _rand(g, 8, H, d, d, scale=0.3)
+    da, db = ops.lowrank_tanh_linear(inner.cuda(), 0, w2.cuda(), decay_bias=bias.cuda()), ref.lowrank_tanh_linear(inner, 0, w2, decay_bias=bias)
+    _close(da, db, "float32", "decays", tol=3e-7)
     sa, sb = state.clone().cuda(), state.clone()
-    a = ops.wkv_scan(rkvg.cuda(), z.cuda(), bias.cuda(), u.cuda(), sa, cd, H, d)
-    b = ref.wkv_scan(rkvg, z, bias, u, sb, cc, H, d)
+    a = ops.wkv_scan(rkvg.cuda(), da, u.cuda(), sa, cd, H, d)
+    b = ref.wkv_scan(rkvg, db, u, sb, cc, H, d)
     _close(a, b, "float32", "read-outs", tol=1e-5)
     _close(sa, sb, "float32", "states", tol=1e-5)
     assert torch.equal(sa[7].cpu(), state[7])                     # a slot of no request in the step

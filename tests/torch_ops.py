@@ -625,8 +625,9 @@ class TorchOps:
             return y, residual
         return y, s.float()
 
-    def lowrank_tanh_linear(self, aw, column, w2):
-        return (torch.tanh(aw[:, column:].double()) @ w2.double().T).float()
+    def lowrank_tanh_linear(self, aw, column, w2, decay_bias=None):
+        z = torch.tanh(aw[:, column:].double()) @ w2.double().T
+        return (z if decay_bias is None else torch.exp(-torch.exp(z + decay_bias.double()))).float()
 
     def general_delta_scan(self, proj, aw, a_bias, z, w_bias, decay_limit, S_all, ctx, H, d, unit_eps):
         T, n = proj.shape[0], H * d
@@ -738,10 +739,10 @@ class TorchOps:
             last[slot] = h[hi - 1].float()
         return torch.stack([h.double() + (before - h.double()) * mu[i].double() for i in range(mu.shape[0])]).to(h.dtype)
 
-    def wkv_scan(self, rkvg, z, w_bias, u, S_all, ctx, H, d):
+    def wkv_scan(self, rkvg, decay, u, S_all, ctx, H, d):
         T = rkvg.shape[1]
         r, k, v = (rkvg[i].double().view(T, H, d) for i in range(3))
-        decay = torch.exp(-torch.exp(z.double() + w_bias.double())).view(T, H, d)
+        decay = decay.double().view(T, H, d)
         bonus = u.double().view(H, d)
         o = torch.zeros((T, H, d), dtype=torch.float64)
         for lo, hi, slot, pos0 in self._requests(ctx):
