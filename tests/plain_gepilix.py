@@ -118,7 +118,7 @@ def window_attention_mixer(h, m: dict, W, p: str) -> torch.Tensor:
 
 # ----------------------------------------------------------------------------- recurrences
 def causal_conv(x, w, b) -> torch.Tensor:
-    """x [T, C], w [C, taps] (last column: the current token), zeros before the start."""
+    """x [T, C], w [C, taps]: y_t = b + sum_j w[:, j] x_(t - taps + 1 + j), with x_s = 0 for s < 0."""
     T, C = x.shape
     n = w.shape[1]
     padded = torch.cat([torch.zeros(n - 1, C, dtype=F), x])
