@@ -52,7 +52,7 @@ __device__ __forceinline__ float tn_norm(float s, float alpha, float w, float b)
 
 // The sum and the norm of four neighbours whose output is `o`.
 template <typename T>
-__device__ __forceinline__ void tn_finish4(const TanhNormArgs& p, int m, int r, int i, float4 o, bool have, float4 res) {
+__device__ __forceinline__ void tn_finish4(const TanhNormArgs& p, int m, int i, float4 o, bool have, float4 res) {
   float4 s = res;
   if (have) {
     if (p.scale) {
@@ -104,7 +104,7 @@ add_tanh_norm_kernel(const A* __restrict__ x, const TanhNormArgs p, int vec_ok) 
           o = make_float4(fmaf(wk[u], v[u].x, o.x), fmaf(wk[u], v[u].y, o.y), fmaf(wk[u], v[u].z, o.z), fmaf(wk[u], v[u].w, o.w));
       }
     }
-    tn_finish4<T>(p, m, r, i, o, have, res);
+    tn_finish4<T>(p, m, i, o, have, res);
     return;
   }
   for (int i = blockIdx.y * 1024 + threadIdx.x; i < min(p.width, (int)(blockIdx.y + 1) * 1024); i += 256) {
@@ -168,7 +168,7 @@ members_tanh_norm_kernel(const A* __restrict__ a0, const A* __restrict__ a1, con
         const float4 wb = *reinterpret_cast<const float4*>(w1 + i);
         o = make_float4(fmaf(v[n].x * r1, wb.x, o.x), fmaf(v[n].y * r1, wb.y, o.y), fmaf(v[n].z * r1, wb.z, o.z), fmaf(v[n].w * r1, wb.w, o.w));
       }
-      tn_finish4<T>(p, m, r, i, o, true, res[n]);
+      tn_finish4<T>(p, m, i, o, true, res[n]);
     }
   } else {
     for (int i = threadIdx.x; i < p.width; i += 256) {
